@@ -10,7 +10,8 @@ execution of a layer that asks for them, and fixed-size state per slot.
 * A group whose mixers read only a *window* of the most recent keys holds only the pages that
   the window still touches: before a step, the pages of a sequence that lie wholly below
   ``length - window + 1`` go back to the group's pool (no query of this or a later step reads
-  them), so such a group can be given a smaller pool (``window_step_tokens``).
+  them), so such a group can be given a smaller pool (``window_step_tokens``).  The same goes for a group whose
+  mixers read only the current *chunk* of positions: pages wholly below the chunk of the step's first position go back.
 * A group of kind "pooled" keeps, beside the window's pages, one row per kv head for every complete
   block of ``pool`` positions (the mean of the block's keys, and of its values) in pages of a second pool;
   those rows stay as long as the sequence lives.
@@ -41,7 +42,9 @@ class KVRequest:
     the pages that no query can reach any more are given back while the sequence grows, except
     those that hold any of the first ``keep_first`` keys (a window that also keeps the sequence's
     first tokens).  ``value_dim``: the size of a value row where it differs from a key's.  ``pool`` (kind
-    "pooled"): positions per block whose mean key and value are kept once the block is complete."""
+    "pooled"): positions per block whose mean key and value are kept once the block is complete.
+    ``chunk``: the mixer reads the keys of the token's own chunk of so many positions (None: no chunks); pages below
+    the chunk of a step's first position are given back like pages below a window."""
     kv_heads: int
     head_dim: int
     kind: str = "full"
@@ -49,6 +52,12 @@ class KVRequest:
     value_dim: Optional[int] = None
     keep_first: int = 0
     pool: int = 0
+    chunk: Optional[int] = None
+
+    @property
+    def bounded(self) -> bool:
+        """Whether a query reads only part of its sequence, so that pages come free while it grows."""
+        return self.window is not None or self.chunk is not None
 
 
 @dataclass(frozen=True)
@@ -120,8 +129,8 @@ class PagedGroup:
                  dtype: torch.dtype, device: torch.device, window_step_tokens: Optional[int] = None):
         self.request = request
         self.entries = entries
-        if request.window is not None and window_step_tokens is not None:
-            # the window's keys and the step's new tokens, both possibly straddling page borders
+        if request.bounded and window_step_tokens is not None:
+            # the window's (or chunk's) keys and the step's new tokens, both possibly straddling page borders
             per_slot = pages_for(self.window_tokens() + window_step_tokens, PAGE) + 1 + pages_for(request.keep_first, PAGE)
             n_pages = max(1, min(n_pages, n_slots * per_slot))
         self.pages = FreeList(n_pages, "page")
@@ -146,9 +155,9 @@ class PagedGroup:
 
     def reserve(self, slot: int, old_length: int, new_length: int) -> None:
         have = self.slot_pages[slot]
-        if self.request.window is not None:
+        if self.request.bounded:
             # the first key any query of this step (positions old_length and up) or of a later
-            # one reads is old_length - window + 1: whole blocks below it go back to the pool
+            # one reads is old_length - window + 1 (or its chunk's first): whole blocks below it go back to the pool
             keep_from = min(self.first_needed(old_length) // PAGE, len(have))
             kept_first = pages_for(self.request.keep_first, PAGE)      # blocks that hold kept first keys stay
             for b in range(max(self.first_block[slot], kept_first), keep_from):
@@ -164,8 +173,13 @@ class PagedGroup:
             self.dirty.add(slot)
 
     def first_needed(self, old_length: int) -> int:
-        """The first position a step that starts at ``old_length``, or a later one, still reads (with a window)."""
-        return max(0, old_length - self.request.window + 1)
+        """The first position a step that starts at ``old_length``, or a later one, still reads (with a window or chunks)."""
+        first = 0
+        if self.request.window is not None:
+            first = max(first, old_length - self.request.window + 1)
+        if self.request.chunk is not None:
+            first = max(first, old_length // self.request.chunk * self.request.chunk)
+        return first
 
     def grows_at(self, old_length: int) -> bool:
         """Whether a sequence of ``old_length`` tokens needs new storage for one more token (so that a step of single tokens
@@ -173,8 +187,8 @@ class PagedGroup:
         return old_length % PAGE == 0
 
     def window_tokens(self) -> int:
-        """Tokens before a step's first that the group keeps per sequence (with a window)."""
-        return self.request.window
+        """Tokens before a step's first that the group keeps per sequence (with a window or chunks)."""
+        return min(n for n in (self.request.window, self.request.chunk) if n is not None)
 
     def release(self, slot: int) -> None:
         for p in reversed(self.pages_of(slot)):
@@ -223,7 +237,7 @@ class PooledWindowGroup(PagedGroup):
                  dtype: torch.dtype, device: torch.device, window_step_tokens: Optional[int] = None):
         if request.pool < 1:
             raise CacheError(f"a pooled cache needs a block size of at least one position, got {request.pool}")
-        if request.window is None or request.keep_first:
+        if request.window is None or request.keep_first or request.chunk is not None:
             raise CacheError("a pooled cache keeps a window of recent keys and no first keys")
         super().__init__(request, entries, n_pages, n_slots, blocks_per_seq, dtype, device, window_step_tokens)
         P = request.pool

@@ -27,7 +27,9 @@
 // weight of a visible key is sigmoid(score + head_bias[h]), not normalised over the keys; and with either, pooled rows: a second paged cache
 // whose row b holds the mean key and mean value of the positions b * pool .. (b + 1) * pool - 1 and is
 // seen by position p when the whole block lies before p's window, (b + 1) * pool - 1 <= p - window.  The
-// pooled rows are walked first, as units of their own (by the CTA of split 0), then the window's keys.
+// pooled rows are walked first, as units of their own (by the CTA of split 0), then the window's keys.  WEIGHTS = 3: softmax
+// over the keys of the token's own chunk of `chunk` positions (counted from position 0), with a learned bias by distance
+// added to the scaled score, rel[h][min(pos - key, rel_n - 1)], and values of another size VD than the keys.
 #include "common.cuh"
 
 namespace kl {
@@ -79,8 +81,14 @@ __device__ __forceinline__ uint32_t pack_bf16(float lo, float hi) {
     return *reinterpret_cast<uint32_t*>(&v);
 }
 
-// SK keys of one kv head, [SK][HD] (a cache page or half of one), into a swizzled stage: the
-// 16-byte chunk c of key row r lands at chunk c ^ (r & 7) of that row.
+// SK rows of one kv head, [SK][HD] (a cache page or half of one), into a swizzled stage: the
+// 16-byte chunk c of row r lands at chunk c ^ swizzle<HD>(r) of that row (r & 7 where a row fills all banks; shorter rows, of
+// which several fill them, take the bits of r above).
+template <int HD> __device__ __forceinline__ int swizzle(int r) {
+    constexpr int CHUNKS = HD / 8;
+    if constexpr (CHUNKS >= 8) return r & 7;
+    else return (r / (8 / CHUNKS)) & (CHUNKS - 1);
+}
 template <int HD, int THREADS, int SK>
 __device__ __forceinline__ void load_keys(bf16* stage, const bf16* __restrict__ src) {
     constexpr int CHUNKS = HD / 8;                       // 16-byte chunks per row
@@ -90,7 +98,7 @@ __device__ __forceinline__ void load_keys(bf16* stage, const bf16* __restrict__ 
     if constexpr (ROWS_PER_TURN % 8 == 0) {
         // A thread keeps its chunk column; its rows are a multiple of 8 apart, so the swizzle term is
         // the same in every turn and the addresses differ by compile-time constants.
-        const uint32_t dst = smem_addr(stage + r0 * HD + ((c ^ (r0 & 7)) << 3));
+        const uint32_t dst = smem_addr(stage + r0 * HD + ((c ^ swizzle<HD>(r0)) << 3));
         const bf16* from = src + r0 * HD + (c << 3);
 #pragma unroll
         for (int t = 0; t < SK / ROWS_PER_TURN; ++t)
@@ -101,7 +109,7 @@ __device__ __forceinline__ void load_keys(bf16* stage, const bf16* __restrict__ 
         for (int t = 0; t < SK / ROWS_PER_TURN; ++t) {
             const int r = r0 + t * ROWS_PER_TURN;
             asm volatile("cp.async.cg.shared.global [%0], [%1], 16;"
-                         ::"r"(smem_addr(stage + r * HD + ((c ^ (r & 7)) << 3))), "l"(src + r * HD + (c << 3)) : "memory");
+                         ::"r"(smem_addr(stage + r * HD + ((c ^ swizzle<HD>(r)) << 3))), "l"(src + r * HD + (c << 3)) : "memory");
         }
     }
 }
@@ -131,6 +139,9 @@ struct AttentionExtra {
     const int* pool_table;        // [slots][pool_blocks_per_seq]
     int pool_blocks_per_seq;
     int pool;                     // positions per block; 0: no pooled rows
+    int chunk;                    // WEIGHTS = 3: positions per chunk; 0: none
+    const float* rel;             // WEIGHTS = 3: float32 [H][rel_n], or null
+    int rel_n;
 };
 
 // The decode step's token of one sequence, for one kv group: its q (the group's G heads) into q_sm
@@ -250,7 +261,7 @@ __device__ __forceinline__ void make_token_qkv(const DecodeFuse& fuse, bf16* q_s
 // SK: keys per stage, a cache page (64) or half of one.  Half pages with two warps make a CTA of the
 // decode layout light enough (48 KB of stages at a head size of 128) for four of them on an SM, or
 // with two stages (32 KB) for six.
-template <int HD, int WM, int WN, int NS, int SK, int WEIGHTS>
+template <int HD, int VD, int WM, int WN, int NS, int SK, int WEIGHTS>
 __global__ void __launch_bounds__(32 * WM * WN, SK < PAGE ? (NS == 2 ? 6 : 4) : (NS == 2 ? ((HD == 64 && WN > 1) ? 4 : 3) : 2))   // half pages: six CTAs of two stages or four of three; whole pages, NS = 2: three CTAs per SM (168 registers, 3 x 64 KB of stages), four in the decode layout with a head size of 64
 attention_mma_kernel(const bf16* __restrict__ q, int q_stride, bf16* __restrict__ out,
                      const bf16* __restrict__ k_cache, const bf16* __restrict__ v_cache,
@@ -270,10 +281,10 @@ attention_mma_kernel(const bf16* __restrict__ q, int q_stride, bf16* __restrict_
     static_assert(PAGE % SK == 0 && KPW % 16 == 0, "attention_mma_kernel: keys per stage and warp");
     constexpr int NT = KPW / 8;                          // score tiles (8 keys each) per warp
     constexpr int KS = HD / 16;                          // k steps of q . k
-    constexpr int ON = HD / 8;                           // output tiles (8 dims each)
+    constexpr int ON = VD / 8;                           // output tiles (8 dims each)
     extern __shared__ __align__(128) uint8_t smem_raw[];
     bf16* k_stage = reinterpret_cast<bf16*>(smem_raw);                   // [NS][SK][HD]
-    bf16* v_stage = k_stage + NS * SK * HD;                              // [NS][SK][HD]
+    bf16* v_stage = k_stage + NS * SK * HD;                              // [NS][SK][VD]
 
     const int b = blockIdx.y;
     const int g = blockIdx.z % KV, z = blockIdx.z / KV;
@@ -302,36 +313,49 @@ attention_mma_kernel(const bf16* __restrict__ q, int q_stride, bf16* __restrict_
         head[i] = g * G + hh;
         pos[i] = valid[i] ? start + tl : -1;
         lo[i] = (window > 0 && valid[i]) ? max(0, pos[i] - window + 1) : 0;
-        nb[i] = (WEIGHTS != 0 && ex.pool > 0 && valid[i]) ? lo[i] / ex.pool : 0;  // pooled rows this row sees: blocks wholly before its window
+        if (WEIGHTS == 3 && ex.chunk > 0 && valid[i]) lo[i] = max(lo[i], pos[i] / ex.chunk * ex.chunk);
+        nb[i] = ((WEIGHTS == 1 || WEIGHTS == 2) && ex.pool > 0 && valid[i]) ? lo[i] / ex.pool : 0;  // pooled rows this row sees: blocks wholly before its window
         hbias[i] = (WEIGHTS == 1 && ex.head_bias != nullptr && valid[i]) ? ex.head_bias[head[i]] * 1.4426950408889634f : 0.f;
     }
     // pages this CTA reads
     const int last_tok = min(T, t0 + BT) - 1;
     const int max_pos = start + last_tok;
-    const int min_lo = window > 0 ? max(0, start + t0 - window + 1) : 0;
+    int min_lo = window > 0 ? max(0, start + t0 - window + 1) : 0;
+    if (WEIGHTS == 3 && ex.chunk > 0) min_lo = max(min_lo, (start + t0) / ex.chunk * ex.chunk);
+    const int max_lo = (WEIGHTS == 3 && ex.chunk > 0) ? max_pos / ex.chunk * ex.chunk : 0;      // keys >= this lie in every row's chunk
+    // the row of the bias table of each of this thread's two rows, and what every far key gets
+    const float* rel[2] = {nullptr, nullptr};
+    float rel_far[2] = {0.f, 0.f};
+    if (WEIGHTS == 3 && ex.rel != nullptr) {
+#pragma unroll
+        for (int i = 0; i < 2; ++i) {
+            rel[i] = ex.rel + (size_t)(valid[i] ? head[i] : 0) * ex.rel_n;
+            rel_far[i] = rel[i][ex.rel_n - 1] * 1.4426950408889634f;
+        }
+    }
     const int first_page = min_lo / PAGE, n_pages = max_pos / PAGE - first_page + 1;
     const int per = (n_pages + S - 1) / S;
     const int p_begin = first_page + z * per, p_end = min(first_page + n_pages, p_begin + per);
     const int* table = block_table + (size_t)slot * blocks_per_seq;
     const int full_below = start + t0;                   // keys <= this are visible to every valid row (no window)
     // Pooled rows: the first PU units of the walk, taken by the CTA of split 0.
-    const int max_nb = (WEIGHTS != 0 && ex.pool > 0) ? max(0, max_pos - window + 1) / ex.pool : 0;
-    const int PU = (WEIGHTS != 0 && ex.pool > 0 && z == 0) ? (max_nb + SK - 1) / SK : 0;
-    const int* ptable = (WEIGHTS != 0 && ex.pool > 0) ? ex.pool_table + (size_t)slot * ex.pool_blocks_per_seq : nullptr;
+    const int max_nb = ((WEIGHTS == 1 || WEIGHTS == 2) && ex.pool > 0) ? max(0, max_pos - window + 1) / ex.pool : 0;
+    const int PU = ((WEIGHTS == 1 || WEIGHTS == 2) && ex.pool > 0 && z == 0) ? (max_nb + SK - 1) / SK : 0;
+    const int* ptable = ((WEIGHTS == 1 || WEIGHTS == 2) && ex.pool > 0) ? ex.pool_table + (size_t)slot * ex.pool_blocks_per_seq : nullptr;
 
     // Units of SK keys this CTA reads: its pages, without what lies wholly behind the last position.
     const int u_begin = p_begin * UPP, u_end = min(p_end * UPP, max_pos / SK + 1);
     // `unit` counts from u_begin - PU: the pooled units come first (their index below u_begin), then the keys' units.
     auto issue = [&](int unit, int st) {
-        if (WEIGHTS != 0 && unit < u_begin) {
+        if ((WEIGHTS == 1 || WEIGHTS == 2) && unit < u_begin) {
             const int pu = unit - (u_begin - PU);
             const size_t off = (((size_t)ptable[pu / UPP] * KV + g) * PAGE + (pu % UPP) * SK) * HD;
             load_keys<HD, THREADS, SK>(k_stage + st * SK * HD, ex.pool_k + off);
-            load_keys<HD, THREADS, SK>(v_stage + st * SK * HD, ex.pool_v + off);
+            load_keys<VD, THREADS, SK>(v_stage + st * SK * VD, ex.pool_v + off);          // pooled rows: VD == HD
         } else {
-            const size_t off = (((size_t)table[unit / UPP] * KV + g) * PAGE + (unit % UPP) * SK) * HD;
-            load_keys<HD, THREADS, SK>(k_stage + st * SK * HD, k_cache + off);
-            load_keys<HD, THREADS, SK>(v_stage + st * SK * HD, v_cache + off);
+            const size_t row = ((size_t)table[unit / UPP] * KV + g) * PAGE + (unit % UPP) * SK;
+            load_keys<HD, THREADS, SK>(k_stage + st * SK * HD, k_cache + row * HD);
+            load_keys<VD, THREADS, SK>(v_stage + st * SK * VD, v_cache + row * VD);
         }
         cp_async_commit();
     };
@@ -404,12 +428,12 @@ attention_mma_kernel(const bf16* __restrict__ q, int q_stride, bf16* __restrict_
     }
     for (int pi = w_begin; pi < u_end; ++pi) {
         const int st = (pi - w_begin) % NS;
-        const bool pooled = WEIGHTS != 0 && pi < u_begin;    // a unit of block means: row index = block index
+        const bool pooled = (WEIGHTS == 1 || WEIGHTS == 2) && pi < u_begin;    // a unit of block means: row index = block index
         if (next < u_end) { issue(next, (next - w_begin) % NS); ++next; } else cp_async_commit();
         cp_async_wait<NS - 1>();                         // all but the NS - 1 newest groups: unit pi has landed
         __syncthreads();
         const bf16* ks_ = k_stage + st * SK * HD;
-        const bf16* vs_ = v_stage + st * SK * HD;
+        const bf16* vs_ = v_stage + st * SK * VD;
         const int key0 = (pooled ? pi - w_begin : pi) * SK + warp_n * KPW;         // first key (or pooled row) of this warp's share
         float s[NT][4];
 #pragma unroll
@@ -422,13 +446,14 @@ attention_mma_kernel(const bf16* __restrict__ q, int q_stride, bf16* __restrict_
                     const int r = warp_n * KPW + n2 * 16 + (lane & 7) + ((lane >> 4) << 3);
                     const int c = ks * 2 + ((lane >> 3) & 1);
                     uint32_t b0, b1, b2, b3;
-                    ldmatrix_x4(smem_addr(ks_ + r * HD + ((c ^ (r & 7)) << 3)), b0, b1, b2, b3);
+                    ldmatrix_x4(smem_addr(ks_ + r * HD + ((c ^ swizzle<HD>(r)) << 3)), b0, b1, b2, b3);
                     mma_bf16(s[2 * n2], qa[ks], b0, b1);
                     mma_bf16(s[2 * n2 + 1], qa[ks], b2, b3);
                 }
             }
             // scale, mask, online softmax
-            const bool need_mask = pooled || key0 + KPW - 1 > full_below || window > 0 || !valid[0] || !valid[1];
+            const bool need_mask = pooled || key0 + KPW - 1 > full_below || window > 0 || key0 < max_lo || !valid[0] || !valid[1];
+            const bool near = WEIGHTS == 3 && ex.rel != nullptr && full_below - (key0 + KPW - 1) < ex.rel_n - 1;    // some pair is nearer than the table's last column
             float mx[2] = {-INFINITY, -INFINITY};
 #pragma unroll
             for (int n = 0; n < NT; ++n) {
@@ -436,6 +461,11 @@ attention_mma_kernel(const bf16* __restrict__ q, int q_stride, bf16* __restrict_
                 for (int c = 0; c < 4; ++c) {
                     const int i = c >> 1;
                     float v = s[n][c] * scale_log2;
+                    if constexpr (WEIGHTS == 3) {
+                        float bias = rel_far[i];
+                        if (near) bias = __ldg(rel[i] + min(max(pos[i] - (key0 + n * 8 + 2 * tq + (c & 1)), 0), ex.rel_n - 1)) * 1.4426950408889634f;
+                        v += bias;
+                    }
                     if (need_mask) {
                         const int kp = key0 + n * 8 + 2 * tq + (c & 1);
                         if (pooled ? kp >= nb[i] : (kp > pos[i] || kp < lo[i])) v = -INFINITY;
@@ -490,7 +520,7 @@ attention_mma_kernel(const bf16* __restrict__ q, int q_stride, bf16* __restrict_
                     const int r = warp_n * KPW + kk * 16 + (lane & 7) + (((lane >> 3) & 1) << 3);
                     const int c = n2 * 2 + (lane >> 4);
                     uint32_t b0, b1, b2, b3;
-                    ldmatrix_x4_trans(smem_addr(vs_ + r * HD + ((c ^ (r & 7)) << 3)), b0, b1, b2, b3);
+                    ldmatrix_x4_trans(smem_addr(vs_ + r * VD + ((c ^ swizzle<VD>(r)) << 3)), b0, b1, b2, b3);
                     mma_bf16(o[2 * n2], pa, b0, b1);
                     mma_bf16(o[2 * n2 + 1], pa, b2, b3);
                 }
@@ -505,7 +535,7 @@ attention_mma_kernel(const bf16* __restrict__ q, int q_stride, bf16* __restrict_
     }
     if constexpr (WN > 1) {
         // merge the warps that shared the rows: through shared memory (the stages are free now)
-        constexpr int OS = HD + 8;                                   // row stride of sm_o: rows 8 banks apart
+        constexpr int OS = VD + 8;                                   // row stride of sm_o: rows 8 banks apart
         float* sm_m = reinterpret_cast<float*>(smem_raw);            // [WN][ROWS]
         float* sm_l = sm_m + WN * ROWS;                              // [WN][ROWS]
         float* sm_o = sm_l + WN * ROWS;                              // [WN][ROWS][OS]
@@ -520,8 +550,8 @@ attention_mma_kernel(const bf16* __restrict__ q, int q_stride, bf16* __restrict_
         }
         __syncthreads();
         const int n_rows = min(BT, T - t0) * Gp;                     // rows of the tile that belong to tokens
-        for (int item = threadIdx.x; item < n_rows * (HD / 4); item += THREADS) {
-            const int r = item / (HD / 4), d = (item % (HD / 4)) * 4;
+        for (int item = threadIdx.x; item < n_rows * (VD / 4); item += THREADS) {
+            const int r = item / (VD / 4), d = (item % (VD / 4)) * 4;
             const int tl = t0 + r / Gp, hh = r % Gp;
             if (hh >= G) continue;
             float M = -INFINITY;
@@ -540,15 +570,15 @@ attention_mma_kernel(const bf16* __restrict__ q, int q_stride, bf16* __restrict_
             const size_t orow = (size_t)(row0 + tl) * H + (g * G + hh);
             if (S == 1) {
                 float inv = 1.f;
-                if constexpr (WEIGHTS == 0) inv = 1.f / L;
+                if constexpr (WEIGHTS == 0 || WEIGHTS == 3) inv = 1.f / L;
                 if constexpr (WEIGHTS == 2) {
                     float keep = 1.f, add = 0.f;
                     if (ex.sink != nullptr) sink_terms(M, ex.sink[g * G + hh] * 1.4426950408889634f, keep, add);
                     inv = keep / (L * keep + add);
                 }
-                *reinterpret_cast<uint2*>(out + orow * HD + d) = make_uint2(pack_bf16(acc.x * inv, acc.y * inv), pack_bf16(acc.z * inv, acc.w * inv));
+                *reinterpret_cast<uint2*>(out + orow * VD + d) = make_uint2(pack_bf16(acc.x * inv, acc.y * inv), pack_bf16(acc.z * inv, acc.w * inv));
             } else {
-                *reinterpret_cast<float4*>(part_o + (orow * S + z) * HD + d) = acc;
+                *reinterpret_cast<float4*>(part_o + (orow * S + z) * VD + d) = acc;
                 if (d == 0) *reinterpret_cast<float2*>(part_ml + (orow * S + z) * 2) = make_float2(M, L);
             }
         }
@@ -567,8 +597,8 @@ attention_mma_kernel(const bf16* __restrict__ q, int q_stride, bf16* __restrict_
                 __threadfence();
                 // four output elements per thread and turn; eight pieces are requested at a time and merged
                 // into a running maximum, sum and output, in ascending order
-                for (int item = threadIdx.x; item < G * (HD / 4); item += THREADS) {
-                    const int hh = item / (HD / 4), d = (item % (HD / 4)) * 4;
+                for (int item = threadIdx.x; item < G * (VD / 4); item += THREADS) {
+                    const int hh = item / (VD / 4), d = (item % (VD / 4)) * 4;
                     const size_t orow = (size_t)row0 * H + (g * G + hh);
                     float M = -INFINITY, L = 0.f;
                     float4 acc = make_float4(0.f, 0.f, 0.f, 0.f);
@@ -579,7 +609,7 @@ attention_mma_kernel(const bf16* __restrict__ q, int q_stride, bf16* __restrict_
                         for (int zz = 0; zz < 8; ++zz) {
                             const bool in = z0 + zz < S;
                             ml[zz] = in ? __ldcg(reinterpret_cast<const float2*>(part_ml + (orow * S + z0 + zz) * 2)) : make_float2(-INFINITY, 0.f);
-                            po[zz] = in ? __ldcg(reinterpret_cast<const float4*>(part_o + (orow * S + z0 + zz) * HD + d)) : make_float4(0.f, 0.f, 0.f, 0.f);
+                            po[zz] = in ? __ldcg(reinterpret_cast<const float4*>(part_o + (orow * S + z0 + zz) * VD + d)) : make_float4(0.f, 0.f, 0.f, 0.f);
                         }
                         float Mc = M;
 #pragma unroll
@@ -595,7 +625,7 @@ attention_mma_kernel(const bf16* __restrict__ q, int q_stride, bf16* __restrict_
                         M = Mc;
                     }
                     const float inv = 1.f / L;
-                    *reinterpret_cast<uint2*>(out + orow * HD + d) = make_uint2(pack_bf16(acc.x * inv, acc.y * inv), pack_bf16(acc.z * inv, acc.w * inv));
+                    *reinterpret_cast<uint2*>(out + orow * VD + d) = make_uint2(pack_bf16(acc.x * inv, acc.y * inv), pack_bf16(acc.z * inv, acc.w * inv));
                 }
             }
         }
@@ -606,7 +636,7 @@ attention_mma_kernel(const bf16* __restrict__ q, int q_stride, bf16* __restrict_
             const size_t orow = (size_t)tok[i] * H + head[i];
             if (S == 1) {
                 float inv = 1.f;
-                if constexpr (WEIGHTS == 0) inv = 1.f / l[i];
+                if constexpr (WEIGHTS == 0 || WEIGHTS == 3) inv = 1.f / l[i];
                 if constexpr (WEIGHTS == 2) {
                     float keep = 1.f, add = 0.f;
                     if (ex.sink != nullptr) sink_terms(m[i], ex.sink[head[i]] * 1.4426950408889634f, keep, add);
@@ -614,11 +644,11 @@ attention_mma_kernel(const bf16* __restrict__ q, int q_stride, bf16* __restrict_
                 }
 #pragma unroll
                 for (int n = 0; n < ON; ++n)
-                    *reinterpret_cast<uint32_t*>(out + orow * HD + n * 8 + 2 * tq) = pack_bf16(o[n][2 * i] * inv, o[n][2 * i + 1] * inv);
+                    *reinterpret_cast<uint32_t*>(out + orow * VD + n * 8 + 2 * tq) = pack_bf16(o[n][2 * i] * inv, o[n][2 * i + 1] * inv);
             } else {
 #pragma unroll
                 for (int n = 0; n < ON; ++n)
-                    *reinterpret_cast<float2*>(part_o + (orow * S + z) * HD + n * 8 + 2 * tq) = make_float2(o[n][2 * i], o[n][2 * i + 1]);
+                    *reinterpret_cast<float2*>(part_o + (orow * S + z) * VD + n * 8 + 2 * tq) = make_float2(o[n][2 * i], o[n][2 * i + 1]);
                 if (tq == 0) { part_ml[(orow * S + z) * 2] = m[i]; part_ml[(orow * S + z) * 2 + 1] = l[i]; }
             }
         }
@@ -626,17 +656,17 @@ attention_mma_kernel(const bf16* __restrict__ q, int q_stride, bf16* __restrict_
 }
 
 // Merge the pieces of a split sequence: maxima and sums are in the exp2 domain of the kernel above.
-template <int HD>
+template <int VD>
 __global__ void attention_mma_combine_kernel(const float* __restrict__ part_o, const float* __restrict__ part_ml,
                                              bf16* __restrict__ out, int H, int S, const float* __restrict__ sink, int weights) {
     pdl_launch_dependents();
     pdl_wait();
     const size_t orow = (size_t)blockIdx.x * H + blockIdx.y;
     if (weights == 1) {                                  // sigmoid weights are not normalised: the pieces add up
-        for (int d = threadIdx.x; d < HD; d += blockDim.x) {
+        for (int d = threadIdx.x; d < VD; d += blockDim.x) {
             float acc = 0.f;
-            for (int z = 0; z < S; ++z) acc += part_o[(orow * S + z) * HD + d];
-            out[orow * HD + d] = __float2bfloat16_rn(acc);
+            for (int z = 0; z < S; ++z) acc += part_o[(orow * S + z) * VD + d];
+            out[orow * VD + d] = __float2bfloat16_rn(acc);
         }
         return;
     }
@@ -644,19 +674,19 @@ __global__ void attention_mma_combine_kernel(const float* __restrict__ part_o, c
     for (int z = 0; z < S; ++z) M = fmaxf(M, part_ml[(orow * S + z) * 2]);
     float keep = 1.f, add = 0.f;
     if (sink != nullptr) sink_terms(M, sink[blockIdx.y] * 1.4426950408889634f, keep, add);
-    for (int d = threadIdx.x; d < HD; d += blockDim.x) {
+    for (int d = threadIdx.x; d < VD; d += blockDim.x) {
         float L = 0.f, acc = 0.f;
         for (int z = 0; z < S; ++z) {
             const float mz = part_ml[(orow * S + z) * 2];
             const float c = mz == -INFINITY ? 0.f : exp2f(mz - M);
             L += part_ml[(orow * S + z) * 2 + 1] * c;
-            acc += part_o[(orow * S + z) * HD + d] * c;
+            acc += part_o[(orow * S + z) * VD + d] * c;
         }
-        out[orow * HD + d] = __float2bfloat16_rn(acc * keep / (L * keep + add));
+        out[orow * VD + d] = __float2bfloat16_rn(acc * keep / (L * keep + add));
     }
 }
 
-template <int HD, int WM, int WN, int NS, int SK = PAGE, int WEIGHTS = 0>
+template <int HD, int WM, int WN, int NS, int SK = PAGE, int WEIGHTS = 0, int VD = HD>
 static int launch_mma(const bf16* q, int q_stride, bf16* out, const bf16* k, const bf16* v, const int* table, int bps,
                       const int* cu, const int* slots, const int* starts, const int* news, float* po, float* pml,
                       int n_seqs, int max_new, int n_rows, int H, int KV, float scale, int window, int S,
@@ -669,20 +699,20 @@ static int launch_mma(const bf16* q, int q_stride, bf16* out, const bf16* k, con
     const int BT = ROWS / Gp;
     const dim3 grid((max_new + BT - 1) / BT, n_seqs, KV * S);
     if (grid.y > 65535 || grid.z > 65535) return KL_ERR_BAD_SIZE;
-    size_t smem = (size_t)2 * NS * SK * HD * sizeof(bf16);
-    if (WN > 1) smem = max(smem, (size_t)(2 * WN * ROWS + WN * ROWS * (HD + 8)) * sizeof(float));
+    size_t smem = (size_t)NS * SK * (HD + VD) * sizeof(bf16);
+    if (WN > 1) smem = max(smem, (size_t)(2 * WN * ROWS + WN * ROWS * (VD + 8)) * sizeof(float));
     static bool configured = false;
     if (!configured) {
-        KL_CUDA(cudaFuncSetAttribute(attention_mma_kernel<HD, WM, WN, NS, SK, WEIGHTS>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem));
+        KL_CUDA(cudaFuncSetAttribute(attention_mma_kernel<HD, VD, WM, WN, NS, SK, WEIGHTS>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem));
         // all of the SM's memory as shared memory: the kernel's data come through cp.async, and how many CTAs fit decides its speed
-        KL_CUDA(cudaFuncSetAttribute(attention_mma_kernel<HD, WM, WN, NS, SK, WEIGHTS>, cudaFuncAttributePreferredSharedMemoryCarveout, (int)cudaSharedmemCarveoutMaxShared));
+        KL_CUDA(cudaFuncSetAttribute(attention_mma_kernel<HD, VD, WM, WN, NS, SK, WEIGHTS>, cudaFuncAttributePreferredSharedMemoryCarveout, (int)cudaSharedmemCarveoutMaxShared));
         configured = true;
     }
-    launch_kernel(attention_mma_kernel<HD, WM, WN, NS, SK, WEIGHTS>, grid, 32 * WM * WN, smem, stream, q, q_stride, out, k, v, table, bps, cu, slots,
+    launch_kernel(attention_mma_kernel<HD, VD, WM, WN, NS, SK, WEIGHTS>, grid, 32 * WM * WN, smem, stream, q, q_stride, out, k, v, table, bps, cu, slots,
         starts, news, po, pml, H, KV, Gp, scale * 1.4426950408889634f, window, S, fuse, ex);
     KL_LAUNCH_CHECK();
     if (S > 1 && !fuse.enabled) {
-        launch_kernel(attention_mma_combine_kernel<HD>, dim3(n_rows, H), HD <= 64 ? 32 : 64, 0, stream, po, pml, out, H, S, ex.sink, WEIGHTS == 1 ? 1 : 0);
+        launch_kernel(attention_mma_combine_kernel<VD>, dim3(n_rows, H), VD <= 64 ? 32 : 64, 0, stream, po, pml, out, H, S, ex.sink, WEIGHTS == 1 ? 1 : 0);
         KL_LAUNCH_CHECK();
     }
     return KL_OK;
@@ -775,12 +805,47 @@ KL_API int kl_attention_mma_extra(const void* q, int q_stride, void* out, const 
     return launch_mma<HD, WM, WN, 2, PAGE, W>((const bf16*)q, q_stride, (bf16*)out, (const bf16*)k_cache, (const bf16*)v_cache,  \
                                               block_table, blocks_per_seq, cu_tokens, seq_slots, seq_starts, seq_new, part_o,   \
                                               part_ml, n_seqs, max_new, n_rows, H, KV, scale, window, splits, none, stream, ex)
+    ex.chunk = 0; ex.rel = nullptr; ex.rel_n = 0;
     // template parameter: 1 = sigmoid weights, 2 = softmax with the options compiled in
     if (hd == 128 && weights == 0) { if (few_rows) KL_MMAX(128, 1, 4, 2); else KL_MMAX(128, 4, 1, 2); }
     if (hd == 128 && weights == 1) { if (few_rows) KL_MMAX(128, 1, 4, 1); else KL_MMAX(128, 4, 1, 1); }
     if (hd == 64 && weights == 0) { if (few_rows) KL_MMAX(64, 1, 4, 2); else KL_MMAX(64, 4, 1, 2); }
     if (hd == 64 && weights == 1) { if (few_rows) KL_MMAX(64, 1, 4, 1); else KL_MMAX(64, 4, 1, 1); }
 #undef KL_MMAX
+    return KL_ERR_BAD_SIZE;
+}
+
+// The same over chunks of `chunk` positions (0: none) with a bias by distance (rel: float32 [H, rel_n], or null) and values of size vd
+// in a cache of their own row size; key and value sizes of 32, 64 and 128.
+KL_API int kl_attention_mma_chunked(const void* q, int q_stride, void* out, const void* k_cache, const void* v_cache,
+                                    const int* block_table, int blocks_per_seq, const int* cu_tokens, const int* seq_slots,
+                                    const int* seq_starts, const int* seq_new, float* part_o, float* part_ml, int n_seqs,
+                                    int max_new, int n_rows, int H, int KV, int hd, int vd, float scale, int window, int splits,
+                                    int few_rows, int chunk, const float* rel, int rel_n, cudaStream_t stream) {
+    if (n_seqs <= 0 || max_new <= 0) return KL_OK;
+    if (KV <= 0 || H % KV || splits < 1 || chunk < 0 || (rel != nullptr && rel_n < 1)) return KL_ERR_BAD_SIZE;
+    if (splits > 1 && (part_o == nullptr || part_ml == nullptr)) return KL_ERR_BAD_SIZE;
+    if (q_stride % 2 || ((uintptr_t)q & 3)) return KL_ERR_BAD_ALIGN;
+    DecodeFuse none;
+    memset(&none, 0, sizeof(none));
+    AttentionExtra ex;
+    memset(&ex, 0, sizeof(ex));
+    ex.chunk = chunk; ex.rel = rel; ex.rel_n = rel_n;
+#define KL_MMAC(HD, VD, WM, WN)                                                                                                     \
+    return launch_mma<HD, WM, WN, 2, PAGE, 3, VD>((const bf16*)q, q_stride, (bf16*)out, (const bf16*)k_cache, (const bf16*)v_cache, \
+                                                  block_table, blocks_per_seq, cu_tokens, seq_slots, seq_starts, seq_new, part_o,  \
+                                                  part_ml, n_seqs, max_new, n_rows, H, KV, scale, window, splits, none, stream, ex)
+#define KL_MMAC_VD(HD)                                                                                     \
+    do {                                                                                                   \
+        if (vd == 32) { if (few_rows) KL_MMAC(HD, 32, 1, 4); else KL_MMAC(HD, 32, 4, 1); }                 \
+        if (vd == 64) { if (few_rows) KL_MMAC(HD, 64, 1, 4); else KL_MMAC(HD, 64, 4, 1); }                 \
+        if (vd == 128) { if (few_rows) KL_MMAC(HD, 128, 1, 4); else KL_MMAC(HD, 128, 4, 1); }              \
+    } while (0)
+    if (hd == 32) KL_MMAC_VD(32);
+    if (hd == 64) KL_MMAC_VD(64);
+    if (hd == 128) KL_MMAC_VD(128);
+#undef KL_MMAC_VD
+#undef KL_MMAC
     return KL_ERR_BAD_SIZE;
 }
 

@@ -16,7 +16,9 @@
 // Options beyond KuiperLLama's attention: values of another size than the keys (`vd` columns of rows
 // that are `v_ld` apart; with v_cache == k_cache and v_ld == hd the values are the leading columns of
 // the keys, which is what attention over a shared latent reads), and a sink: a learned number per
-// head that joins the softmax's denominator as exp(sink) and has no value.
+// head that joins the softmax's denominator as exp(sink) and has no value; chunks: a token reads the keys of its own chunk
+// of `chunk` positions, counted from position 0; and a learned bias by distance: rel[h, min(pos - key, rel_n - 1)] is
+// added to the scaled score.
 #include "common.cuh"
 
 namespace kl {
@@ -67,7 +69,8 @@ attention_simt_kernel(const T* __restrict__ q, int q_stride, T* __restrict__ out
                       const T* __restrict__ k_cache, const T* __restrict__ v_cache,
                       const int* __restrict__ block_table, int blocks_per_seq,
                       const int* __restrict__ positions, const int* __restrict__ token_slot,
-                      int H, int KV, int hd, float scale, int window, int vd, int v_ld, const float* __restrict__ sink) {
+                      int H, int KV, int hd, float scale, int window, int vd, int v_ld, const float* __restrict__ sink, int chunk,
+                      const float* __restrict__ rel, int rel_n) {
     pdl_launch_dependents();
     pdl_wait();
     extern __shared__ float smem[];
@@ -87,7 +90,8 @@ attention_simt_kernel(const T* __restrict__ q, int q_stride, T* __restrict__ out
     for (int i = threadIdx.x; i < hd; i += blockDim.x) q_s[i] = to_f32(qrow[i]);
     __syncthreads();
 
-    const int lo = window > 0 ? max(0, pos - window + 1) : 0;
+    int lo = window > 0 ? max(0, pos - window + 1) : 0;
+    if (chunk > 0) lo = max(lo, pos / chunk * chunk);
     float m = -INFINITY, l = 0.f;
     float acc[PL];
 #pragma unroll
@@ -101,7 +105,10 @@ attention_simt_kernel(const T* __restrict__ q, int q_stride, T* __restrict__ out
         const int key = base + lane;
         const bool valid = key >= lo && key <= pos;
         float s = -INFINITY;
-        if (valid) s = dot_row<T>(k_cache + page_off + (size_t)lane * hd, q_s, hd) * scale;
+        if (valid) {
+            s = dot_row<T>(k_cache + page_off + (size_t)lane * hd, q_s, hd) * scale;
+            if (rel != nullptr) s += rel[(size_t)h * rel_n + min(pos - key, rel_n - 1)];
+        }
         const float m_new = fmaxf(m, warp_max(s));                   // finite: the chunk holds a valid key
         const float corr = expf(m - m_new);                          // exp(-inf) = 0 at the first chunk
         const float p = valid ? expf(s - m_new) : 0.f;
@@ -154,15 +161,15 @@ attention_simt_kernel(const T* __restrict__ q, int q_stride, T* __restrict__ out
 using namespace kl;
 
 // q: rows of q_stride elements, head h at column h * hd.  out: [tokens, H * vd].  vd <= 0 means values like
-// keys (vd = v_ld = hd).  sink: float32 [H] or null.
+// keys (vd = v_ld = hd).  sink: float32 [H] or null.  chunk: positions per chunk (0: none).  rel: float32 [H, rel_n] or null.
 KL_API int kl_attention_simt(const void* q, int q_stride, void* out, const void* k_cache, const void* v_cache,
                              const int* block_table, int blocks_per_seq, const int* positions,
                              const int* token_slot, int n_tokens, int H, int KV, int hd, float scale, int window,
-                             int vd, int v_ld, const float* sink, int dtype, cudaStream_t stream) {
+                             int vd, int v_ld, const float* sink, int chunk, const float* rel, int rel_n, int dtype, cudaStream_t stream) {
     if (n_tokens <= 0) return KL_OK;
     if (vd <= 0) { vd = hd; v_ld = hd; }
     if (vd > ATT_MAX_VALUE_DIM || hd <= 0 || v_ld < vd || KV <= 0 || H % KV) return KL_ERR_BAD_SIZE;
-    if (H > 65535) return KL_ERR_BAD_SIZE;
+    if (H > 65535 || chunk < 0 || (rel != nullptr && rel_n < 1)) return KL_ERR_BAD_SIZE;
     const dim3 grid(n_tokens, H);
     const size_t smem = (size_t)(hd + 2 * ATT_WARPS + ATT_WARPS * vd) * sizeof(float);
     if (smem > 200 * 1024) return KL_ERR_BAD_SIZE;
@@ -171,7 +178,7 @@ KL_API int kl_attention_simt(const void* q, int q_stride, void* out, const void*
         if (smem > 48 * 1024) KL_CUDA(cudaFuncSetAttribute(attention_simt_kernel<T, PL>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem)); \
         launch_kernel(attention_simt_kernel<T, PL>, grid, ATT_WARPS * 32, smem, stream, (const T*)q, q_stride, (T*)out,       \
                       (const T*)k_cache, (const T*)v_cache, block_table, blocks_per_seq, positions, token_slot, H, KV, hd,    \
-                      scale, window, vd, v_ld, sink);                                                                         \
+                      scale, window, vd, v_ld, sink, chunk, rel, rel_n);                                                                         \
     } while (0)
     if (dtype == KL_F32) { if (vd <= 256) KL_ATT(float, 8); else KL_ATT(float, 16); }
     else if (dtype == KL_BF16) { if (vd <= 256) KL_ATT(bf16, 8); else KL_ATT(bf16, 16); }

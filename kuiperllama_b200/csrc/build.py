@@ -44,6 +44,7 @@ SOURCES: Dict[str, str] = {
     "linear_recurrence": "linear_recurrence.cu",
     "short_conv": "short_conv.cu",
     "outer_recurrence": "outer_recurrence.cu",
+    "mlstm": "mlstm.cu",
     "attention_mixed": "attention_mixed.cu",
     "attention_mixed_tiled": "attention_mixed_tiled.cu",
     "qk_prepare": "qk_prepare.cu",

@@ -64,9 +64,11 @@ struct GemmArgs {
     const int* tile_group;
     int group_rows;
     // With swiglu and act_custom: min(g, limit) * sigmoid(alpha * min(g, limit)) * (clamp(u, -limit, limit) + shift),
-    // no clamp when limit <= 0 (act_custom 0: silu(g) * u).
+    // no clamp when limit <= 0 (act_custom 0: silu(g) * u).  With act_cubic c the sigmoid's argument is
+    // alpha * g * (1 + c g^2): with alpha = 2 sqrt(2 / pi) and c = 0.044715 that is the tanh form of gelu, since
+    // (1 + tanh(y)) / 2 = sigmoid(2 y).
     int act_custom;
-    float act_limit, act_alpha, act_shift;
+    float act_limit, act_alpha, act_shift, act_cubic;
     // The plain epilogue's activation on a complete result in bfloat16 (grouped products, no k cuts): 0 none, 1 the
     // squared relu max(y, 0)^2.
     int act_plain;
@@ -97,7 +99,7 @@ __device__ __forceinline__ float plain_act(const GemmArgs& args, float y) {
 __device__ __forceinline__ float gated_mul(const GemmArgs& args, float g, float u) {
     if (!args.act_custom) return silu_mul(g, u);
     if (args.act_limit > 0.f) { g = fminf(g, args.act_limit); u = fminf(fmaxf(u, -args.act_limit), args.act_limit); }
-    return __fdividef(g, 1.0f + __expf(-args.act_alpha * g)) * (u + args.act_shift);
+    return __fdividef(g, 1.0f + __expf(-args.act_alpha * g * fmaf(args.act_cubic * g, g, 1.0f))) * (u + args.act_shift);
 }
 
 // The squared relu on 32 accumulator columns in place.
@@ -718,6 +720,12 @@ static int launch_pairs(const CUtensorMap& ma, const CUtensorMap& mb, const Gemm
     return KL_OK;
 }
 
+// The gated epilogue by name: 0 none, 1 silu(g) * u, 2 gelu(g) * u in its tanh form.
+static void set_gated(GemmArgs& args, int kind) {
+    args.swiglu = kind != 0;
+    if (kind == 2) { args.act_custom = 1; args.act_limit = 0.f; args.act_alpha = 1.5957691216057308f; args.act_shift = 0.f; args.act_cubic = 0.044715f; }
+}
+
 static bool aligned_operand(const void* p, long long ld, int K) {
     return ((uintptr_t)p & 15) == 0 && (ld % 8) == 0 && (K % 8) == 0 && K > 0;
 }
@@ -727,11 +735,12 @@ static bool aligned_operand(const void* p, long long ld, int K) {
 using namespace kl;
 
 // out[M, N] = a[M, K] * w[N, K]^T, tokens as tile rows (any M).  out is bf16 (out_f32 = 0) or
-// float32.  Needs 16-byte aligned bases and row strides (K % 8 == 0): else KL_ERR_BAD_ALIGN.
+// float32.  Needs 16-byte aligned bases and row strides (K % 8 == 0): else KL_ERR_BAD_ALIGN.  swiglu: 0 plain, 1 silu(gate) * up,
+// 2 gelu(gate) * up (see set_gated).
 KL_API int kl_gemm_tcgen05(const void* a, long long lda, const void* w, long long ldw, void* out, long long ldo, int M,
                            int N, int K, int out_f32, int swiglu, int* status, cudaStream_t stream) {
     if (M <= 0 || N <= 0) return KL_OK;
-    if (swiglu && (out_f32 || N % 128)) return KL_ERR_BAD_SIZE;
+    if (swiglu < 0 || swiglu > 2 || (swiglu && (out_f32 || N % 128))) return KL_ERR_BAD_SIZE;
     if (!aligned_operand(a, lda, K) || !aligned_operand(w, ldw, K)) return KL_ERR_BAD_ALIGN;
     CUtensorMap ma, mb;
     int rc;
@@ -745,11 +754,13 @@ KL_API int kl_gemm_tcgen05(const void* a, long long lda, const void* w, long lon
         const int tiles_m2 = (M + 2 * TC_BM - 1) / (2 * TC_BM), tiles_n2 = (N + 255) / 256;
         if ((long long)tiles_m2 * tiles_n2 > 0x3fffffffLL) return KL_ERR_BAD_SIZE;
         GemmArgs pargs{out, ldo, 0, M, N, (K + TC_BK - 1) / TC_BK, out_f32, status, tiles_m2, tiles_n2, swiglu};
+        set_gated(pargs, swiglu);
         return launch_pairs(ma, mb, pargs, 2 * min(tiles_m2 * tiles_n2, sms2 / 2), stream);
     }
     if ((rc = make_map(&mb, w, N, K, ldw, 256)) != KL_OK) return rc;
     const int tiles_m = (M + TC_BM - 1) / TC_BM, tiles_n = (N + 255) / 256;
     GemmArgs args{out, ldo, 0, M, N, (K + TC_BK - 1) / TC_BK, out_f32, status, tiles_m, tiles_n, swiglu};
+    set_gated(args, swiglu);
     if ((long long)tiles_m * tiles_n > 0x7fffffffLL) return KL_ERR_BAD_SIZE;
     const int sms = kl::sm_count();
     if (sms <= 0) return KL_ERR_SETUP;
@@ -838,7 +849,7 @@ KL_API int kl_gemm_tcgen05_skinny(const void* a, long long lda, const void* w, l
     if (M <= 0 || N <= 0) return KL_OK;
     if (M > 512) return KL_ERR_BAD_SIZE;
     if (M > 64 && (scale_ss != nullptr || sink != nullptr)) return KL_ERR_BAD_SIZE;     // the folded norm: one tile of tokens
-    if (swiglu && (splits != 1 || out_f32 || N % 128)) return KL_ERR_BAD_SIZE;
+    if (swiglu < 0 || swiglu > 2 || (swiglu && (splits != 1 || out_f32 || N % 128))) return KL_ERR_BAD_SIZE;
     if (!aligned_operand(w, ldw, K) || !aligned_operand(a, lda, K)) return KL_ERR_BAD_ALIGN;
     if (scale_ss != nullptr && scale_ss_n < 1) return KL_ERR_BAD_SIZE;
     if (sink != nullptr && (!out_f32 || swiglu || sink_ss == nullptr || sink_counters == nullptr || ldo != N ||
@@ -857,6 +868,7 @@ KL_API int kl_gemm_tcgen05_skinny(const void* a, long long lda, const void* w, l
     const int token_tiles = (M + bn - 1) / bn;
     GemmArgs args{out, ldo, (long long)M * ldo, N, M, k_blocks, out_f32, status, token_tiles, 0, swiglu,
                   scale_ss, scale_ss_n, scale_eps, K, sink, sink_ss, sink_counters, sink_w, (__nv_bfloat16*)sink_scaled};
+    set_gated(args, swiglu);
     dim3 grid(((N + TC_BM - 1) / TC_BM) * token_tiles, 1, splits);
     // A grid of at most one CTA per SM (small matrices) gives each CTA the whole of the SM's shared
     // memory as stages: what a CTA has in flight bounds what it streams (96 KB over the 1.5 us a tile

@@ -3,7 +3,8 @@
 //   moe_route_kernel    a warp per token: s = softmax(z) over all experts in 32 bits (z plus a bias per expert
 //                       where one is given), the `top` largest (the lower index among equals), their scores
 //                       as weights (divided by their sum if asked, which is the softmax over the chosen
-//                       logits alone).
+//                       logits alone).  Or s = sigmoid(z), with a correction per expert that joins the scores for
+//                       the choice but not for the weights; weights times a scale.
 //   moe_plan_kernel     one CTA: counts per expert, a list of (token, choice) pairs sorted by expert in
 //                       which every expert's run is padded to whole tiles, the expert of every tile, and
 //                       each pair's place in the list.  Everything stays on the device, so a step with
@@ -22,22 +23,31 @@ constexpr int MOE_MAX_PER_LANE = 8;      // experts <= 256
 constexpr int MOE_PLAN_THREADS = 1024;
 constexpr int MOE_MAX_EXPERTS = 32 * MOE_MAX_PER_LANE;
 
+struct RouteArgs {
+    const float* logits; long long ld;
+    const float* bias;              // [experts], joins the logits, or null
+    const float* correction;        // [experts], joins the scores for the choice alone, or null
+    int tokens, experts, top, renormalise, groups, keep_groups, sigmoid, group_top;    // group_top: a group's score is the sum of its so many best
+    float renorm_eps, scale;
+    int* choice; float* weight;
+};
+
 __global__ void __launch_bounds__(128)
-moe_route_kernel(const float* __restrict__ logits, long long ld, const float* __restrict__ bias, int tokens, int experts, int top, int renormalise,
-                 int groups, int keep_groups, float renorm_eps, int* __restrict__ choice, float* __restrict__ weight) {
+moe_route_kernel(const RouteArgs A) {
     pdl_launch_dependents();
     pdl_wait();
     __shared__ float group_best[4][MOE_MAX_EXPERTS];
     const int lane = threadIdx.x & 31;
     const int t = blockIdx.x * 4 + (threadIdx.x >> 5);
-    if (t >= tokens) return;
-    const float* z = logits + (size_t)t * ld;
-    float s[MOE_MAX_PER_LANE];
+    if (t >= A.tokens) return;
+    const int experts = A.experts, top = A.top, groups = A.groups;
+    const float* z = A.logits + (size_t)t * A.ld;
+    float s[MOE_MAX_PER_LANE], w[MOE_MAX_PER_LANE];          // choice scores (taken and absent experts hold -inf) and weights
     float m = -INFINITY;
 #pragma unroll
     for (int i = 0; i < MOE_MAX_PER_LANE; ++i) {
         const int e = lane + 32 * i;
-        s[i] = e < experts ? (bias ? z[e] + bias[e] : z[e]) : -INFINITY;
+        s[i] = e < experts ? (A.bias ? z[e] + A.bias[e] : z[e]) : -INFINITY;
         m = fmaxf(m, s[i]);
     }
     m = warp_max(m);
@@ -45,26 +55,42 @@ moe_route_kernel(const float* __restrict__ logits, long long ld, const float* __
 #pragma unroll
     for (int i = 0; i < MOE_MAX_PER_LANE; ++i) {
         const int e = lane + 32 * i;
-        s[i] = e < experts ? expf(s[i] - m) : -1.f;          // taken and absent experts hold -1: below every score
-        sum += e < experts ? s[i] : 0.f;
+        w[i] = 0.f;
+        if (e < experts) {
+            w[i] = A.sigmoid ? 1.0f / (1.0f + expf(-s[i])) : expf(s[i] - m);
+            s[i] = A.correction ? w[i] + A.correction[e] : w[i];
+            sum += w[i];
+        }
     }
-    sum = warp_sum(sum);
-    if (groups > 1 && keep_groups < groups) {
-        // Experts form `groups` equal groups of neighbours; a group's score is its largest score, and only the experts
-        // of the `keep_groups` best groups (the lower index among equals) stay in the choice.
+    sum = A.sigmoid ? 1.f : warp_sum(sum);                   // softmax: scores are w / sum
+    float* weight = A.weight + (size_t)t * top;
+    if (groups > 1 && A.keep_groups < groups) {
+        // Experts form `groups` equal groups of neighbours; a group's score is its largest choice score, or the sum of its
+        // `group_top` largest, and only the experts of the `keep_groups` best groups (the lower index among equals) stay.
         float* gb = group_best[threadIdx.x >> 5];
         const int per = experts / groups;
-        for (int g = lane; g < groups; g += 32) gb[g] = -1.f;
-        __syncwarp();
         for (int g = 0; g < groups; ++g) {
-            float b = -1.f;
+            float total = 0.f, below = INFINITY;             // the largest not above `below`, each expert once
+            int after = -1;
+            for (int k = 0; k < min(A.group_top, per); ++k) {
+                float b = -INFINITY;
+                int be = 0x7fffffff;
 #pragma unroll
-            for (int i = 0; i < MOE_MAX_PER_LANE; ++i) {
-                const int e = lane + 32 * i;
-                if (e < experts && e / per == g) b = fmaxf(b, s[i]);
+                for (int i = 0; i < MOE_MAX_PER_LANE; ++i) {
+                    const int e = lane + 32 * i;
+                    if (e < experts && e / per == g && (s[i] < below || (s[i] == below && e > after)) && (s[i] > b || (s[i] == b && e < be))) { b = s[i]; be = e; }
+                }
+#pragma unroll
+                for (int o = 16; o > 0; o >>= 1) {
+                    const float ob = __shfl_xor_sync(0xffffffffu, b, o);
+                    const int oe = __shfl_xor_sync(0xffffffffu, be, o);
+                    if (ob > b || (ob == b && oe < be)) { b = ob; be = oe; }
+                }
+                total += b;
+                below = b;
+                after = be;
             }
-            b = warp_max(b);
-            if (lane == 0) gb[g] = b;
+            if (lane == 0) gb[g] = total;
         }
         __syncwarp();
         // rank of every group: how many groups come before it (a larger score, or an equal one with a lower index)
@@ -76,14 +102,14 @@ moe_route_kernel(const float* __restrict__ logits, long long ld, const float* __
                 const float mine_b = gb[g];
                 int before = 0;
                 for (int o = 0; o < groups; ++o) before += (gb[o] > mine_b || (gb[o] == mine_b && o < g)) ? 1 : 0;
-                if (before >= keep_groups) s[i] = -1.f;
+                if (before >= A.keep_groups) s[i] = -INFINITY;
             }
         }
     }
     float chosen_sum = 0.f, mine = 0.f;
     int mine_e = 0;
     for (int k = 0; k < top; ++k) {
-        float best = -1.f;
+        float best = -INFINITY;
         int best_e = 0x7fffffff;
 #pragma unroll
         for (int i = 0; i < MOE_MAX_PER_LANE; ++i)
@@ -94,20 +120,23 @@ moe_route_kernel(const float* __restrict__ logits, long long ld, const float* __
             const int oe = __shfl_xor_sync(0xffffffffu, best_e, o);
             if (ob > best || (ob == best && oe < best_e)) { best = ob; best_e = oe; }
         }
+        if (best_e >= experts) best_e = k;                   // no comparable score is left (logits that are not numbers): any expert, in bounds
+        float chosen_w = 0.f;
 #pragma unroll
         for (int i = 0; i < MOE_MAX_PER_LANE; ++i)
-            if (lane + 32 * i == best_e) s[i] = -1.f;
-        chosen_sum += best;
-        if (lane == k % 32) { mine = best; mine_e = best_e; }
+            if (lane + 32 * i == best_e) { chosen_w = w[i]; s[i] = -INFINITY; }
+        chosen_w = __shfl_sync(0xffffffffu, chosen_w, best_e & 31);
+        chosen_sum += chosen_w;
+        if (lane == k % 32) { mine = chosen_w; mine_e = best_e; }
         if (k % 32 == 31 || k == top - 1) {
             const int kk = (k / 32) * 32 + lane;
-            if (kk <= k) { choice[(size_t)t * top + kk] = mine_e; weight[(size_t)t * top + kk] = mine; }
+            if (kk <= k) { A.choice[(size_t)t * top + kk] = mine_e; weight[kk] = mine; }
         }
     }
-    // weights: the softmax scores, or those divided by the chosen ones' sum
+    // weights: the scores, or those divided by the chosen ones' sum, times the scale
     __syncwarp();
-    const float denom = renormalise ? chosen_sum + renorm_eps * sum : sum;      // scores s = exp / sum: s_k / (sum of chosen s + eps)
-    for (int kk = lane; kk < top; kk += 32) weight[(size_t)t * top + kk] = weight[(size_t)t * top + kk] / denom;
+    const float denom = A.renormalise ? chosen_sum + A.renorm_eps * sum : sum;      // softmax scores are w / sum: s_k / (sum of chosen s + eps)
+    for (int kk = lane; kk < top; kk += 32) weight[kk] = weight[kk] / denom * A.scale;
 }
 
 __global__ void __launch_bounds__(MOE_PLAN_THREADS)
@@ -200,13 +229,17 @@ KL_API int kl_moe_gather(const void* x, long long ld, const int* list_rows, int 
     return KL_OK;
 }
 
+// scores: 0 softmax over the experts, 1 sigmoid; correction: float32 [experts] or null; group_top: see RouteArgs.
 KL_API int kl_moe_route(const float* logits, long long ld, const float* bias, int tokens, int experts, int top, int renormalise, int groups,
-                        int keep_groups, float renorm_eps, int* choice, float* weight, cudaStream_t stream) {
+                        int keep_groups, float renorm_eps, int scores, const float* correction, int group_top, float scale,
+                        int* choice, float* weight, cudaStream_t stream) {
     if (tokens <= 0) return KL_OK;
     if (experts <= 0 || experts > MOE_MAX_EXPERTS || top <= 0 || top > experts) return KL_ERR_BAD_SIZE;
     if (groups < 1 || experts % groups || keep_groups < 1 || keep_groups > groups || top > keep_groups * (experts / groups)) return KL_ERR_BAD_SIZE;
-    launch_kernel(moe_route_kernel, (tokens + 3) / 4, 128, 0, stream, logits, ld, bias, tokens, experts, top, renormalise, groups, keep_groups,
-                  renorm_eps, choice, weight);
+    if ((scores != 0 && scores != 1) || group_top < 1) return KL_ERR_BAD_SIZE;
+    const RouteArgs A{logits, ld, bias, correction, tokens, experts, top, renormalise, groups, keep_groups, scores, group_top, renorm_eps, scale,
+                      choice, weight};
+    launch_kernel(moe_route_kernel, (tokens + 3) / 4, 128, 0, stream, A);
     KL_LAUNCH_CHECK();
     return KL_OK;
 }

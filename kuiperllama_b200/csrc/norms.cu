@@ -17,7 +17,8 @@
 // (rmsnorm_kernel.cu:70-106) and its add as a kernel of its own (add_kernel.cu:4-12).
 //
 // A second kernel is the per-head RMS norm with an output gate that linear-attention mixers
-// end with: out[t, h, :] = x[t, h, :] / rms(x[t, h, :]) * w * silu(gate[t, h, :]).
+// end with: out[t, h, :] = x[t, h, :] / rms(x[t, h, :]) * w * silu(gate[t, h, :]) (or sigmoid; x may first be divided by a
+// number per head).
 #include "common.cuh"
 
 namespace kl {
@@ -236,13 +237,17 @@ norm_chain_kernel(float* __restrict__ residual, const T* __restrict__ delta, lon
     for (int i = threadIdx.x; i < hidden; i += blockDim.x) o[i] = from_f32<T>(buf[i]);
 }
 
+// The gate's factor: silu(a), or sigmoid(a) where `sigmoid` is set.
+__device__ __forceinline__ float gate_factor(float a, int sigmoid) { return (sigmoid ? 1.0f : a) / (1.0f + expf(-a)); }
+
 // x: float32 [tokens, heads * dim]; gate: compute dtype, row stride gate_ld, same columns;
-// w: float32 [dim] shared by the heads (or null).  One warp per (token, head).
+// w: float32 [dim] shared by the heads (or null); divisor: float32 [tokens, heads] (or null), what a head is divided by
+// first.  One warp per (token, head).
 template <typename T>
 __global__ void __launch_bounds__(128)
 head_rmsnorm_gate_kernel(const float* __restrict__ x, const T* __restrict__ gate, long long gate_ld, const float* __restrict__ w,
                          T* __restrict__ out, long long out_ld, float out_scale, int tokens, int heads, int dim, float eps, int gate_first,
-                         int wide_weight) {
+                         int wide_weight, const float* __restrict__ divisor, int sigmoid) {
     pdl_launch_dependents();
     pdl_wait();
     const int lane = threadIdx.x & 31;
@@ -253,32 +258,31 @@ head_rmsnorm_gate_kernel(const float* __restrict__ x, const T* __restrict__ gate
     const T* g = gate ? gate + (size_t)t * gate_ld + (size_t)h * dim : nullptr;
     const float* wr = w != nullptr ? w + (wide_weight ? (size_t)h * dim : 0) : nullptr;
     T* o = out + (size_t)t * out_ld + (size_t)h * dim;
+    const float pre = divisor != nullptr ? 1.0f / divisor[(size_t)t * heads + h] : 1.0f;
     if (gate_first && g != nullptr) {
         // the gate comes before the norm: y = x silu(g), then y / rms(y) * w
         float ss = 0.f;
         for (int i = lane; i < dim; i += 32) {
-            const float a = to_f32(g[i]);
-            const float y = xr[i] * (a / (1.0f + expf(-a)));
+            const float y = xr[i] * pre * gate_factor(to_f32(g[i]), sigmoid);
             ss += y * y;
         }
         ss = warp_sum(ss);
         const float inv = 1.0f / sqrtf(ss / (float)dim + eps);
         for (int i = lane; i < dim; i += 32) {
-            const float a = to_f32(g[i]);
-            float y = xr[i] * (a / (1.0f + expf(-a))) * inv;
+            float y = xr[i] * pre * gate_factor(to_f32(g[i]), sigmoid) * inv;
             if (wr != nullptr) y *= wr[i];
             o[i] = from_f32<T>(y * out_scale);
         }
         return;
     }
     float ss = 0.f;
-    for (int i = lane; i < dim; i += 32) ss += xr[i] * xr[i];
+    for (int i = lane; i < dim; i += 32) { const float y = xr[i] * pre; ss += y * y; }
     ss = warp_sum(ss);
-    const float inv = 1.0f / sqrtf(ss / (float)dim + eps);
+    const float inv = pre / sqrtf(ss / (float)dim + eps);
     for (int i = lane; i < dim; i += 32) {
         float y = xr[i] * inv;
         if (wr != nullptr) y *= wr[i];
-        if (g != nullptr) { const float a = to_f32(g[i]); y *= a / (1.0f + expf(-a)); }
+        if (g != nullptr) y *= gate_factor(to_f32(g[i]), sigmoid);
         o[i] = from_f32<T>(y * out_scale);
     }
 }
@@ -288,7 +292,7 @@ template <typename T>
 __global__ void __launch_bounds__(1024)
 head_rmsnorm_gate_block_kernel(const float* __restrict__ x, const T* __restrict__ gate, long long gate_ld, const float* __restrict__ w,
                                T* __restrict__ out, long long out_ld, float out_scale, int heads, int dim, float eps, int gate_first,
-                               int wide_weight) {
+                               int wide_weight, const float* __restrict__ divisor, int sigmoid) {
     pdl_launch_dependents();
     pdl_wait();
     __shared__ float scratch[33];
@@ -298,24 +302,24 @@ head_rmsnorm_gate_block_kernel(const float* __restrict__ x, const T* __restrict_
     const float* wr = w != nullptr ? w + (wide_weight ? (size_t)h * dim : 0) : nullptr;
     T* o = out + (size_t)t * out_ld + (size_t)h * dim;
     const bool first = gate_first && g != nullptr;
+    const float pre = divisor != nullptr ? 1.0f / divisor[(size_t)t * heads + h] : 1.0f;
     float ss = 0.f;
     for (int i = threadIdx.x; i < dim; i += blockDim.x) {
-        float y = xr[i];
-        if (first) { const float a = to_f32(g[i]); y *= a / (1.0f + expf(-a)); }
+        float y = xr[i] * pre;
+        if (first) y *= gate_factor(to_f32(g[i]), sigmoid);
         ss += y * y;
     }
     ss = block_sum(ss, scratch);
     const float inv = 1.0f / sqrtf(ss / (float)dim + eps);
     for (int i = threadIdx.x; i < dim; i += blockDim.x) {
-        float y = xr[i];
+        float y = xr[i] * pre;
         if (first) {
-            const float a = to_f32(g[i]);
-            y = y * (a / (1.0f + expf(-a))) * inv;
+            y = y * gate_factor(to_f32(g[i]), sigmoid) * inv;
             if (wr != nullptr) y *= wr[i];
         } else {
             y *= inv;
             if (wr != nullptr) y *= wr[i];
-            if (g != nullptr) { const float a = to_f32(g[i]); y *= a / (1.0f + expf(-a)); }
+            if (g != nullptr) y *= gate_factor(to_f32(g[i]), sigmoid);
         }
         o[i] = from_f32<T>(y * out_scale);
     }
@@ -430,16 +434,17 @@ KL_API int kl_norm_chain(float* residual, const void* delta, long long delta_ld,
 }
 
 KL_API int kl_head_rmsnorm_gate(const float* x, const void* gate, long long gate_ld, const float* w, void* out, long long out_ld,
-                                float out_scale, int tokens, int heads, int dim, float eps, int gate_first, int wide_weight, int dtype,
+                                float out_scale, int tokens, int heads, int dim, float eps, int gate_first, int wide_weight,
+                                const float* divisor, int sigmoid, int dtype,
                                 cudaStream_t stream) {
     if (tokens <= 0 || heads <= 0) return KL_OK;
     if (dim <= 0) return KL_ERR_BAD_SIZE;
     const long long items = (long long)tokens * heads;
     if (dim >= 512) {
         if (dtype == KL_F32)
-            launch_kernel(head_rmsnorm_gate_block_kernel<float>, (int)items, dim >= 2048 ? 1024 : 256, 0, stream, x, (const float*)gate, gate_ld, w, (float*)out, out_ld, out_scale, heads, dim, eps, gate_first, wide_weight);
+            launch_kernel(head_rmsnorm_gate_block_kernel<float>, (int)items, dim >= 2048 ? 1024 : 256, 0, stream, x, (const float*)gate, gate_ld, w, (float*)out, out_ld, out_scale, heads, dim, eps, gate_first, wide_weight, divisor, sigmoid);
         else if (dtype == KL_BF16)
-            launch_kernel(head_rmsnorm_gate_block_kernel<bf16>, (int)items, dim >= 2048 ? 1024 : 256, 0, stream, x, (const bf16*)gate, gate_ld, w, (bf16*)out, out_ld, out_scale, heads, dim, eps, gate_first, wide_weight);
+            launch_kernel(head_rmsnorm_gate_block_kernel<bf16>, (int)items, dim >= 2048 ? 1024 : 256, 0, stream, x, (const bf16*)gate, gate_ld, w, (bf16*)out, out_ld, out_scale, heads, dim, eps, gate_first, wide_weight, divisor, sigmoid);
         else
             return KL_ERR_BAD_DTYPE;
         KL_LAUNCH_CHECK();
@@ -447,9 +452,9 @@ KL_API int kl_head_rmsnorm_gate(const float* x, const void* gate, long long gate
     }
     const int blocks = (int)((items + 3) / 4);
     if (dtype == KL_F32)
-        launch_kernel(head_rmsnorm_gate_kernel<float>, blocks, 128, 0, stream, x, (const float*)gate, gate_ld, w, (float*)out, out_ld, out_scale, tokens, heads, dim, eps, gate_first, wide_weight);
+        launch_kernel(head_rmsnorm_gate_kernel<float>, blocks, 128, 0, stream, x, (const float*)gate, gate_ld, w, (float*)out, out_ld, out_scale, tokens, heads, dim, eps, gate_first, wide_weight, divisor, sigmoid);
     else if (dtype == KL_BF16)
-        launch_kernel(head_rmsnorm_gate_kernel<bf16>, blocks, 128, 0, stream, x, (const bf16*)gate, gate_ld, w, (bf16*)out, out_ld, out_scale, tokens, heads, dim, eps, gate_first, wide_weight);
+        launch_kernel(head_rmsnorm_gate_kernel<bf16>, blocks, 128, 0, stream, x, (const bf16*)gate, gate_ld, w, (bf16*)out, out_ld, out_scale, tokens, heads, dim, eps, gate_first, wide_weight, divisor, sigmoid);
     else
         return KL_ERR_BAD_DTYPE;
     KL_LAUNCH_CHECK();

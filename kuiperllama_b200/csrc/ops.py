@@ -104,15 +104,19 @@ def _i32(t: Optional[torch.Tensor], name: str) -> None:
 # --------------------------------------------------------------------------- row-wise
 
 def embedding(ids: torch.Tensor, table: torch.Tensor, out: torch.Tensor, error_flag: torch.Tensor,
-              scale: float = 1.0) -> None:
-    """out[t] = scale * float32(table[ids[t]]); ids outside the table set error_flag[0] = 1."""
-    _cuda(ids, table, out, error_flag)
-    _i32(ids, "ids"); _i32(error_flag, "error_flag")
+              scale: float = 1.0, positions: Optional[torch.Tensor] = None, freq: Optional[torch.Tensor] = None) -> None:
+    """out[t] = scale * float32(table[ids[t]]); ids outside the table set error_flag[0] = 1.  With ``freq`` (float32
+    [2, ceil(hidden / 2)]: a frequency per pair, and what its rounding left over) a sinusoid of ``positions`` is added in the
+    same kernel: sin(p f_i) to entry 2i, cos(p f_i) to entry 2i + 1."""
+    _cuda(ids, table, out, error_flag, positions, freq)
+    _i32(ids, "ids"); _i32(error_flag, "error_flag"); _i32(positions, "positions")
     n, (vocab, hidden) = ids.numel(), table.shape
     _need(table.is_contiguous() and out.is_contiguous() and out.dtype == torch.float32, "embedding: bad layout")
     _need(out.shape[0] >= n and out.shape[1] == hidden, "embedding: output shape")
-    _check(lib("rowwise").kl_embedding(_ptr(ids), n, _ptr(table), dtype_code(table.dtype), vocab, hidden,
-                                       ctypes.c_float(scale), _ptr(out), _ptr(error_flag), _stream()), "embedding")
+    _need(freq is None or (positions is not None and positions.numel() >= n and freq.dtype == torch.float32 and freq.is_contiguous()
+                           and tuple(freq.shape) == (2, (hidden + 1) // 2)), "embedding: frequencies [2, pairs] and a position per token")
+    _check(lib("rowwise").kl_embedding(_ptr(ids), n, _ptr(table), dtype_code(table.dtype), vocab, hidden, ctypes.c_float(scale),
+                                       _ptr(positions if freq is not None else None), _ptr(freq), _ptr(out), _ptr(error_flag), _stream()), "embedding")
 
 
 def logit_transform(logits: torch.Tensor, scale: float = 1.0, softcap: float = 0.0) -> None:
@@ -160,13 +164,16 @@ def add_rmsnorm(residual: torch.Tensor, delta: Optional[torch.Tensor], weight: t
                                          dtype_code(out.dtype), _stream()), "add_rmsnorm")
 
 
-def swiglu(gate_up: torch.Tensor, out: torch.Tensor) -> None:
-    """out[t, i] = silu(gate_up[t, i]) * gate_up[t, I + i]."""
+GATED_ACTIVATIONS = {"silu": 1, "gelu_tanh": 2}     # what a gated feed-forward applies to its gate
+
+
+def swiglu(gate_up: torch.Tensor, out: torch.Tensor, activation: str = "silu") -> None:
+    """out[t, i] = act(gate_up[t, i]) * gate_up[t, I + i], act one of ``GATED_ACTIVATIONS``."""
     _cuda(gate_up, out)
     tokens, two_i = gate_up.shape
     _need(two_i % 2 == 0 and out.shape == (tokens, two_i // 2), "swiglu: shapes")
     _need(gate_up.is_contiguous() and out.is_contiguous() and gate_up.dtype == out.dtype, "swiglu: layout")
-    _check(lib("rowwise").kl_swiglu(_ptr(gate_up), _ptr(out), tokens, two_i // 2, dtype_code(out.dtype), _stream()),
+    _check(lib("rowwise").kl_swiglu(_ptr(gate_up), _ptr(out), tokens, two_i // 2, GATED_ACTIVATIONS[activation] - 1, dtype_code(out.dtype), _stream()),
            "swiglu")
 
 
@@ -223,12 +230,18 @@ def norm_chain(residual: torch.Tensor, delta: Optional[torch.Tensor], out: Optio
 
 
 def head_rmsnorm_gate(x: torch.Tensor, gate: Optional[torch.Tensor], weight: Optional[torch.Tensor], out: torch.Tensor,
-                      heads: int, dim: int, eps: float, gate_first: bool = False, out_scale: float = 1.0) -> None:
+                      heads: int, dim: int, eps: float, gate_first: bool = False, out_scale: float = 1.0, *,
+                      divisor: Optional[torch.Tensor] = None, gate_act: str = "silu") -> None:
     """out[t, h, :] = x[t, h, :] / sqrt(mean(x[t, h, :]^2) + eps) * weight * silu(gate[t, h, :]); x float32
     [tokens, heads * dim], gate (compute dtype, any row stride) and weight (float32 [dim], or [heads * dim]: a weight
     per channel) optional.  ``gate_first``: the gate comes before the norm, out = norm(x * silu(gate)) * weight.  ``out`` may
-    be a column slice of a wider matrix; the result is multiplied by ``out_scale`` (in 32 bits, before it is rounded)."""
-    _cuda(x, gate, weight, out)
+    be a column slice of a wider matrix; the result is multiplied by ``out_scale`` (in 32 bits, before it is rounded).
+    ``divisor``: float32 [tokens, heads], what every head of x is divided by before anything else; ``gate_act`` "sigmoid":
+    the gate's factor is sigmoid(gate) instead of silu(gate)."""
+    _cuda(x, gate, weight, out, divisor)
+    _need(gate_act in ("silu", "sigmoid"), f"head_rmsnorm_gate: gate {gate_act!r} (silu, sigmoid)")
+    _need(divisor is None or (divisor.dtype == torch.float32 and divisor.is_contiguous() and divisor.shape[0] >= x.shape[0]
+                              and divisor.shape[1] == heads), "head_rmsnorm_gate: divisor")
     n = x.shape[0]
     _need(x.dtype == torch.float32 and x.is_contiguous() and x.shape[1] == heads * dim, "head_rmsnorm_gate: x")
     _columns(out, n, heads * dim, "head_rmsnorm_gate: out")
@@ -239,7 +252,7 @@ def head_rmsnorm_gate(x: torch.Tensor, gate: Optional[torch.Tensor], weight: Opt
     wide = weight is not None and weight.numel() == heads * dim and heads > 1
     _check(lib("norms").kl_head_rmsnorm_gate(_ptr(x), _ptr(gate), ctypes.c_longlong(gate.stride(0) if gate is not None else 0),
                                              _ptr(weight), _ptr(out), ctypes.c_longlong(out.stride(0)), ctypes.c_float(out_scale), n, heads, dim,
-                                             ctypes.c_float(eps), int(bool(gate_first)), int(wide),
+                                             ctypes.c_float(eps), int(bool(gate_first)), int(wide), _ptr(divisor), int(gate_act == "sigmoid"),
                                              dtype_code(out.dtype), _stream()), "head_rmsnorm_gate")
 
 
@@ -416,11 +429,14 @@ def rope_kv_write(qkv: torch.Tensor, inv_freq: Optional[torch.Tensor], rotary_di
 def attention_simt(q: torch.Tensor, q_stride: int, out: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Tensor,
                    block_table: torch.Tensor, positions: torch.Tensor, token_slot: torch.Tensor, n_tokens: int,
                    num_heads: int, num_kv_heads: int, head_dim: int, scale: float, window: int = 0,
-                   value_dim: Optional[int] = None, sink: Optional[torch.Tensor] = None) -> None:
+                   value_dim: Optional[int] = None, sink: Optional[torch.Tensor] = None, *, chunk: int = 0,
+                   distance_bias: Optional[torch.Tensor] = None) -> None:
     """out[t, h] = softmax(scale * q[t, h] . K[slot_t, lo..pos_t]) V over the paged cache.  ``value_dim``: the
     values are the first so many columns of ``v_cache``'s rows (which may be the key cache itself);
-    ``sink``: float32 [heads], exp(sink[h]) joins head h's denominator."""
-    _cuda(q, out, k_cache, v_cache, block_table, positions, token_slot, sink)
+    ``sink``: float32 [heads], exp(sink[h]) joins head h's denominator; ``chunk``: a token reads the keys of its own chunk of so
+    many positions (0: no chunks); ``distance_bias``: float32 [heads, n], column min(pos - key, n - 1) is added to the score."""
+    _cuda(q, out, k_cache, v_cache, block_table, positions, token_slot, sink, distance_bias)
+    _need_distance_bias(distance_bias, num_heads, chunk)
     _i32(positions, "positions"); _i32(token_slot, "token_slot"); _i32(block_table, "block_table")
     vd = head_dim if value_dim is None else int(value_dim)
     _need(out.is_contiguous() and out.shape[0] >= n_tokens and out.shape[1] == num_heads * vd, "attention: out shape")
@@ -434,8 +450,57 @@ def attention_simt(q: torch.Tensor, q_stride: int, out: torch.Tensor, k_cache: t
     _check(lib("attention_simt").kl_attention_simt(_ptr(q), q_stride, _ptr(out), _ptr(k_cache), _ptr(v_cache),
                                                    _ptr(block_table), block_table.shape[1], _ptr(positions),
                                                    _ptr(token_slot), n_tokens, num_heads, num_kv_heads, head_dim,
-                                                   ctypes.c_float(scale), int(window or 0), vd, int(v_cache.shape[3]), _ptr(sink),
+                                                   ctypes.c_float(scale), int(window or 0), vd, int(v_cache.shape[3]), _ptr(sink), int(chunk or 0),
+                                                   _ptr(distance_bias), 0 if distance_bias is None else distance_bias.shape[1],
                                                    dtype_code(q.dtype), _stream()), "attention_simt")
+
+
+def _need_distance_bias(bias: Optional[torch.Tensor], heads: int, chunk: int) -> None:
+    _need(int(chunk or 0) >= 0, "attention: the chunk size must not be negative")
+    _need(bias is None or (bias.dtype == torch.float32 and bias.is_contiguous() and bias.dim() == 2 and bias.shape[0] == heads
+                           and bias.shape[1] >= 1), "attention: the distance bias is float32 [heads, distances]")
+
+
+def qk_row_prepare(proj: torch.Tensor, q_col: int, k_col: int, v_col: int, q_out: torch.Tensor, step, block_table: Optional[torch.Tensor],
+                   k_cache: Optional[torch.Tensor], v_cache: Optional[torch.Tensor], num_heads: int, num_kv_heads: int, head_dim: int,
+                   value_dim: int, *, norm: bool = True, eps: float = 0.0, q_norm_weight: Optional[torch.Tensor] = None,
+                   k_norm_weight: Optional[torch.Tensor] = None, v_first: Optional[torch.Tensor] = None,
+                   v_lambda: Optional[torch.Tensor] = None, v_keep: Optional[torch.Tensor] = None) -> None:
+    """For every token: q and k over the root mean square of the WHOLE projection (all heads at once, ``eps`` inside the root)
+    times a weight per column; q into ``q_out`` [tokens, H * head_dim] (which may be its columns of ``proj``), k into
+    ``k_cache``; v, or (1 - lambda) v + lambda ``v_first`` [tokens, KV * value_dim] with lambda = ``v_lambda`` (one float32
+    number), into ``v_cache``; v as projected also into ``v_keep`` where given.  ``proj``: rows in the compute dtype, or float32
+    pieces [S, tokens, columns] of a product whose K range was cut.  Both caches None: q (and ``v_keep``) alone."""
+    _cuda(proj, q_out, block_table, k_cache, v_cache, q_norm_weight, k_norm_weight, v_first, v_lambda, v_keep)
+    _i32(block_table, "block_table")
+    H, KV, hd, vd, n = num_heads, num_kv_heads, head_dim, value_dim, step.n_tokens
+    dt = q_out.dtype
+    rows, parts, n_parts, stride = proj, None, 0, 0
+    if _partials(proj):
+        _need(proj.dtype == torch.float32 and proj.is_contiguous(), "qk_row_prepare: pieces must be float32 [S, tokens, columns]")
+        rows, parts, n_parts, stride = None, proj, proj.shape[0], proj.shape[1] * proj.shape[2]
+    else:
+        _need(proj.dtype == dt and proj.dim() == 2 and proj.stride(1) == 1, "qk_row_prepare: projections")
+    ld = proj.stride(-2)
+    _need(proj.shape[-2] >= n and max(q_col + H * hd, k_col + KV * hd, v_col + KV * vd) <= proj.shape[-1], "qk_row_prepare: columns")
+    _columns(q_out, n, H * hd, "qk_row_prepare: q_out")
+    for w, size, name in ((q_norm_weight, H * hd, "q_norm_weight"), (k_norm_weight, KV * hd, "k_norm_weight")):
+        _need(w is None or (w.dtype == torch.float32 and w.is_contiguous() and w.numel() == size), f"qk_row_prepare: {name} must be float32 [{size}]")
+    _need((k_cache is None) == (v_cache is None), "qk_row_prepare: both caches or none")
+    if k_cache is not None:
+        _need(block_table is not None and k_cache.dtype == dt == v_cache.dtype and k_cache.is_contiguous() and v_cache.is_contiguous()
+              and tuple(k_cache.shape[1:]) == (KV, PAGE, hd) and tuple(v_cache.shape[1:]) == (KV, PAGE, vd), "qk_row_prepare: cache layout")
+    _columns(v_first, n, KV * vd, "qk_row_prepare: v_first")
+    _need(v_first is None or (v_first.dtype == dt and v_lambda is not None and v_lambda.dtype == torch.float32 and v_lambda.numel() == 1),
+          "qk_row_prepare: values to mix in need their factor")
+    _need(v_keep is None or (v_keep.dtype == dt and v_keep.is_contiguous() and v_keep.shape[0] >= n and v_keep.shape[1] == KV * vd),
+          "qk_row_prepare: v_keep")
+    _check(lib("qk_prepare").kl_qk_row_prepare(
+        _ptr(rows), _ptr(parts), n_parts, ctypes.c_longlong(stride), ctypes.c_longlong(ld), q_col, k_col, v_col, int(bool(norm)),
+        ctypes.c_float(eps), _ptr(q_norm_weight), _ptr(k_norm_weight), _ptr(q_out), ctypes.c_longlong(q_out.stride(0)), _ptr(k_cache),
+        _ptr(v_cache), _ptr(block_table), 0 if block_table is None else block_table.shape[1], _ptr(v_first),
+        ctypes.c_longlong(v_first.stride(0) if v_first is not None else 0), _ptr(v_lambda), _ptr(v_keep), _ptr(step.positions),
+        _ptr(step.token_slot), n, H, KV, hd, vd, dtype_code(dt), _stream()), "qk_row_prepare")
 
 
 def qk_prepare(proj: torch.Tensor, q_col: int, k_col: int, v_col: Optional[int], positions: torch.Tensor, token_slot: torch.Tensor,
@@ -630,15 +695,25 @@ def grouped_gemv(a: torch.Tensor, w: torch.Tensor, out: torch.Tensor, a_rows: Op
 # --------------------------------------------------------------------------- mixture of experts
 
 MOE_MAX_EXPERTS = 256          # equals MOE_MAX_EXPERTS in moe.cu
+ROUTER_SCORES = {"softmax": 0, "sigmoid": 1}
 
 
 def moe_route(logits: torch.Tensor, top: int, renormalise: bool = False, groups: int = 1, keep_groups: int = 1,
-              renorm_eps: float = 0.0, bias: Optional[torch.Tensor] = None):
+              renorm_eps: float = 0.0, bias: Optional[torch.Tensor] = None, *, scores: str = "softmax",
+              correction: Optional[torch.Tensor] = None, group_top: int = 1, scale: float = 1.0):
     """(choice int32 [tokens, top], weight float32 [tokens, top]) from float32 router logits [tokens, experts]:
     softmax over all experts, the ``top`` largest, their scores (divided by their sum + ``renorm_eps`` if ``renormalise``).
     With ``groups`` > 1 the experts form that many equal groups of neighbours, a group's score is its largest score, and
-    only experts of the ``keep_groups`` best groups can be chosen.  ``bias``: float32 [experts], added to the logits first."""
-    _cuda(logits, bias)
+    only experts of the ``keep_groups`` best groups can be chosen.  ``bias``: float32 [experts], added to the logits first.
+    ``scores`` "sigmoid": every expert's score is sigmoid(z) by itself; ``correction`` (float32 [experts]) joins the scores for
+    the choice, of groups and experts alike, but not for the weights; ``group_top``: a group's score is the sum of its so many
+    best; ``scale`` multiplies the weights."""
+    _cuda(logits, bias, correction)
+    _need(scores in ROUTER_SCORES, f"moe_route: scores {scores!r} ({', '.join(ROUTER_SCORES)})")
+    _need(correction is None or (correction.dtype == torch.float32 and correction.is_contiguous() and correction.numel() == logits.shape[1]),
+          "moe_route: float32 correction per expert")
+    _need(correction is None or scores == "sigmoid", "moe_route: a correction goes with sigmoid scores")
+    _need(group_top >= 1, "moe_route: a group's score takes at least one expert")
     n, E = logits.shape
     _need(bias is None or (bias.dtype == torch.float32 and bias.is_contiguous() and bias.numel() == E), "moe_route: float32 bias per expert")
     _need(logits.dtype == torch.float32 and logits.stride(1) == 1, "moe_route: float32 logits")
@@ -648,7 +723,8 @@ def moe_route(logits: torch.Tensor, top: int, renormalise: bool = False, groups:
     _need(groups >= 1 and E % groups == 0 and 1 <= keep_groups <= groups and top <= keep_groups * (E // groups),
           f"moe_route: {groups} groups of which {keep_groups} are kept do not hold {top} of {E} experts")
     _check(lib("moe").kl_moe_route(_ptr(logits), ctypes.c_longlong(logits.stride(0)), _ptr(bias), n, E, top, int(bool(renormalise)), int(groups),
-                                   int(keep_groups), ctypes.c_float(renorm_eps), _ptr(choice), _ptr(weight), _stream()), "moe_route")
+                                   int(keep_groups), ctypes.c_float(renorm_eps), ROUTER_SCORES[scores], _ptr(correction), int(group_top),
+                                   ctypes.c_float(scale), _ptr(choice), _ptr(weight), _stream()), "moe_route")
     return choice, weight
 
 
@@ -916,13 +992,24 @@ def decay_lowrank(r1: torch.Tensor, W2: torch.Tensor, b: Optional[torch.Tensor],
 
 def outer_recurrence(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, a: torch.Tensor, state: torch.Tensor, y: torch.Tensor, step,
                      heads: int, groups: int, N: int, P: int, c: Optional[torch.Tensor] = None, skip: Optional[torch.Tensor] = None,
-                     q_scale: float = 1.0) -> None:
+                     q_scale: float = 1.0, *, normaliser: Optional[tuple] = None) -> None:
     """S_t = diag(a_t) S_(t-1) + (c_t k_t) v_t^T and y_t = S_t^T (q_scale q_t) + skip v_t per head over a ragged step, from and
     into ``state`` float32 [slots, >= heads * N * P] (S as [heads, N, P]).  ``q``, ``k`` [rows, groups * N] and ``v``
     [rows, heads * P] share one dtype (float32 or the compute dtype) and may be column slices; ``a`` float32 [rows, heads]
     (one decay per head) or [rows, heads * N] (one per row of S); ``c`` float32 [rows, heads] or None; ``skip`` float32
-    [heads] or None; ``y`` float32 [rows, heads * P]."""
+    [heads] or None; ``y`` float32 [rows, heads * P].  ``normaliser`` = (n, floor, den, eps): beside S a vector
+    n_t = diag(a_t) n_(t-1) + c_t k_t per head (``n`` float32 [slots, heads * N], rows as far apart as ``state``'s), and
+    den_t = max(|n_t . q_scale q_t|, floor_t) + eps; ``floor`` and ``den`` float32 [rows, heads]."""
     _cuda(q, k, v, a, state, y, c, skip)
+    n_state = floor = den = None
+    den_eps = 0.0
+    if normaliser is not None:
+        n_state, floor, den, den_eps = normaliser
+        _cuda(n_state, floor, den)
+        _need(n_state.dtype == torch.float32 and n_state.dim() == 2 and n_state.stride(1) == 1 and n_state.stride(0) == state.stride(0)
+              and n_state.shape[1] >= heads * N, "outer_recurrence: the normaliser's state")
+        for t in (floor, den):
+            _need(t.dtype == torch.float32 and t.is_contiguous() and t.shape[0] >= step.n_tokens and t.shape[1] == heads, "outer_recurrence: floor and den")
     n = step.n_tokens
     _columns(q, n, groups * N, "outer_recurrence: q"); _columns(k, n, groups * N, "outer_recurrence: k")
     _columns(v, n, heads * P, "outer_recurrence: v")
@@ -940,7 +1027,31 @@ def outer_recurrence(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, a: torch
         _ptr(q), ctypes.c_longlong(q.stride(0)), 0, _ptr(k), ctypes.c_longlong(k.stride(0)), 0, _ptr(v), ctypes.c_longlong(v.stride(0)), 0,
         _ptr(a), ctypes.c_longlong(a.stride(0)), int(per_row), _ptr(c), ctypes.c_longlong(c.stride(0) if c is not None else 0), _ptr(skip),
         _ptr(state), ctypes.c_longlong(state.stride(0)), _ptr(y), ctypes.c_longlong(y.stride(0)), _ptr(step.cu_tokens),
-        _ptr(step.seq_slots), step.n_seqs, int(step.max_new), heads, groups, N, P, ctypes.c_float(q_scale), dtype_code(q.dtype), _stream()), "outer_recurrence")
+        _ptr(step.seq_slots), step.n_seqs, int(step.max_new), heads, groups, N, P, ctypes.c_float(q_scale), _ptr(n_state), _ptr(floor), _ptr(den),
+        ctypes.c_float(den_eps), dtype_code(q.dtype), _stream()), "outer_recurrence")
+
+
+def mlstm_gates(x: torch.Tensor, weight: torch.Tensor, bias: torch.Tensor, cap: float, state: torch.Tensor, step):
+    """The factors of a matrix memory with exponential gates (see mlstm.cu), float32 [rows, heads] each: (a, c, floor), from the
+    log gates i = cap tanh(z_i / cap) and f = logsigmoid(cap tanh(z_f / cap)) with z = ``weight`` x + ``bias`` in 32 bits, and
+    the running maximum in ``state`` (float32 [slots, >= heads]), which moves on.  ``weight`` [2 * heads, width] in the compute
+    dtype: the input gates' rows, then the forget gates'; ``bias`` float32 [2 * heads]."""
+    _cuda(x, weight, bias, state)
+    n, dev = step.n_tokens, x.device
+    H, width = weight.shape[0] // 2, weight.shape[1]
+    _columns(x, n, width, "mlstm_gates: x")
+    _need(weight.dtype == x.dtype and weight.is_contiguous() and weight.shape[0] == 2 * H, "mlstm_gates: weight [2 heads, width]")
+    _need(bias.dtype == torch.float32 and bias.is_contiguous() and bias.numel() == 2 * H and cap > 0, "mlstm_gates: bias and cap")
+    _need(state.dtype == torch.float32 and state.dim() == 2 and state.stride(1) == 1 and state.shape[1] >= H, "mlstm_gates: state")
+    single = bool(step.is_decode) and n == step.n_seqs
+    # rows that belong to no sequence (a small step's padding) are not written by the scan: keep them defined
+    a, c, floor = (torch.empty if single else torch.ones)((3, n, H), dtype=torch.float32, device=dev).unbind(0)
+    z = None if single else torch.empty((n, 2 * H), dtype=torch.float32, device=dev)
+    _check(lib("mlstm").kl_mlstm_gates(
+        _ptr(x), ctypes.c_longlong(x.stride(0)), _ptr(weight), width, _ptr(bias), ctypes.c_float(cap), _ptr(state),
+        ctypes.c_longlong(state.stride(0)), _ptr(z), _ptr(a), _ptr(c), _ptr(floor), _ptr(step.cu_tokens), _ptr(step.seq_slots), n,
+        step.n_seqs, int(step.max_new), H, int(single), dtype_code(x.dtype), _stream()), "mlstm_gates", 1 if single else 2)
+    return a, c, floor
 
 
 # --------------------------------------------------------------------------- attention with mixed heads
@@ -1175,11 +1286,11 @@ def skinny_splits(N: int, K: int, M: int = 1) -> int:
     return (k_blocks + per - 1) // per
 
 
-def gemm_tcgen05(a: torch.Tensor, w: torch.Tensor, out: torch.Tensor, swiglu: bool = False) -> None:
+def gemm_tcgen05(a: torch.Tensor, w: torch.Tensor, out: torch.Tensor, swiglu: bool = False, activation: str = "silu") -> None:
     """out[M, N] = a @ w^T on the tensor cores, tokens as tile rows (any M; pairs of CTAs on tiles of
     256 tokens where the token count suits, single CTAs on tiles of 128 otherwise).  With ``swiglu``
     the rows of ``w`` alternate 64 gate rows and 64 up rows and out[M, N / 2] receives
-    silu(gate) * up."""
+    act(gate) * up (``activation`` one of ``GATED_ACTIVATIONS``)."""
     _cuda(a, w, out)
     (M, K), (N, K2) = a.shape, w.shape
     _need(K == K2 and out.shape[0] >= M and out.shape[1] == (N // 2 if swiglu else N), "gemm_tcgen05: shapes")
@@ -1187,7 +1298,7 @@ def gemm_tcgen05(a: torch.Tensor, w: torch.Tensor, out: torch.Tensor, swiglu: bo
     _need(_tc_ok(a, w, out), "gemm_tcgen05: operands must be bfloat16 with 16-byte aligned rows")
     _check(lib("gemm_tcgen05").kl_gemm_tcgen05(_ptr(a), ctypes.c_longlong(a.stride(0)), _ptr(w),
                                                ctypes.c_longlong(w.stride(0)), _ptr(out), ctypes.c_longlong(out.stride(0)),
-                                               M, N, K, int(out.dtype == torch.float32), int(swiglu),
+                                               M, N, K, int(out.dtype == torch.float32), GATED_ACTIVATIONS[activation] if swiglu else 0,
                                                _status_ptr(a.device), _stream()), "gemm_tcgen05")
 
 
@@ -1316,11 +1427,11 @@ def gemm_skinny_partials(a: torch.Tensor, w: torch.Tensor, splits: Optional[int]
 
 
 def gemm_skinny(a: torch.Tensor, w: torch.Tensor, out: torch.Tensor, splits: Optional[int] = None,
-                swiglu: bool = False) -> None:
+                swiglu: bool = False, activation: str = "silu") -> None:
     """out[M, N] = a @ w^T for M <= SKINNY_MAX_ROWS tokens: weights as tile rows, each weight read once, the
     K range cut into ``splits`` pieces whose float32 partial sums are added in a fixed order.
     With ``swiglu`` (rows of ``w`` alternate 64 gate and 64 up rows; no cut) out[M, N / 2]
-    receives silu(gate) * up."""
+    receives act(gate) * up (``activation`` one of ``GATED_ACTIVATIONS``)."""
     _cuda(a, w, out)
     (M, K), (N, K2) = a.shape, w.shape
     _need(K == K2 and out.shape[0] >= M and out.shape[1] == (N // 2 if swiglu else N) and M <= SKINNY_MAX_ROWS, "gemm_skinny: shapes")
@@ -1332,8 +1443,8 @@ def gemm_skinny(a: torch.Tensor, w: torch.Tensor, out: torch.Tensor, splits: Opt
     if splits == 1:
         _check(L.kl_gemm_tcgen05_skinny(_ptr(a), ctypes.c_longlong(a.stride(0)), _ptr(w), ctypes.c_longlong(w.stride(0)),
                                         _ptr(out), ctypes.c_longlong(out.stride(0)), M, N, K, 1,
-                                        int(out.dtype == torch.float32), int(swiglu), *_NO_STREAM_FUSION, st, _stream()),
-               "gemm_skinny")
+                                        int(out.dtype == torch.float32), GATED_ACTIVATIONS[activation] if swiglu else 0,
+                                        *_NO_STREAM_FUSION, st, _stream()), "gemm_skinny")
         return
     partial = torch.empty((splits, M, N), dtype=torch.float32, device=a.device)
     _check(L.kl_gemm_tcgen05_skinny(_ptr(a), ctypes.c_longlong(a.stride(0)), _ptr(w), ctypes.c_longlong(w.stride(0)),
@@ -1447,6 +1558,38 @@ def attention_mma(q: torch.Tensor, q_stride: int, out: torch.Tensor, k_cache: to
         "attention_mma", 2 if splits > 1 else 1)
 
 
+CHUNKED_MMA_DIMS = (32, 64, 128)       # key and value sizes of the tensor-core kernel with chunks and a distance bias
+
+
+def attention_chunked_mma(q: torch.Tensor, q_stride: int, out: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Tensor,
+                          block_table: torch.Tensor, step, num_heads: int, num_kv_heads: int, head_dim: int, value_dim: int, scale: float,
+                          *, window: int = 0, chunk: int = 0, distance_bias: Optional[torch.Tensor] = None, splits: int = 1,
+                          few_rows: bool = False) -> None:
+    """Tensor-core softmax attention of ``step`` over the keys of every token's own chunk of ``chunk`` positions (0: no chunks;
+    a ``window`` may cut them further), with ``distance_bias`` (float32 [heads, n]: column min(distance, n - 1) joins the
+    scaled score) and values of ``value_dim`` columns; bfloat16, key and value sizes of 32, 64 and 128, groups of up to 16 heads.
+    ``few_rows`` and ``splits`` as for ``attention_mma``."""
+    _cuda(q, out, k_cache, v_cache, block_table, distance_bias)
+    _i32(block_table, "block_table")
+    H, KV, hd, vd, n = num_heads, num_kv_heads, head_dim, value_dim, step.n_tokens
+    _need(q.dtype == out.dtype == k_cache.dtype == v_cache.dtype == torch.bfloat16, "attention_chunked_mma: bfloat16 only")
+    _need(hd in CHUNKED_MMA_DIMS and vd in CHUNKED_MMA_DIMS, f"attention_chunked_mma: sizes {hd}, {vd} not in {CHUNKED_MMA_DIMS}")
+    _need(out.is_contiguous() and out.shape[0] >= n and out.shape[1] == H * vd, "attention_chunked_mma: out shape")
+    _need(k_cache.is_contiguous() and v_cache.is_contiguous() and tuple(k_cache.shape[1:]) == (KV, PAGE, hd)
+          and tuple(v_cache.shape[1:]) == (KV, PAGE, vd), "attention_chunked_mma: cache layout")
+    _need(H % KV == 0 and H // KV <= 16, "attention_chunked_mma: group size up to 16")
+    _need_distance_bias(distance_bias, H, chunk)
+    po = pml = None
+    if splits > 1:
+        po = torch.empty((n, H, splits, vd), dtype=torch.float32, device=q.device)
+        pml = torch.empty((n, H, splits, 2), dtype=torch.float32, device=q.device)
+    _check(lib("attention_mma").kl_attention_mma_chunked(
+        _ptr(q), q_stride, _ptr(out), _ptr(k_cache), _ptr(v_cache), _ptr(block_table), block_table.shape[1], _ptr(step.cu_tokens),
+        _ptr(step.seq_slots), _ptr(step.seq_starts), _ptr(step.seq_new), _ptr(po), _ptr(pml), step.n_seqs, int(step.max_new), n, H, KV, hd, vd,
+        ctypes.c_float(scale), int(window or 0), splits, int(few_rows), int(chunk or 0), _ptr(distance_bias),
+        0 if distance_bias is None else distance_bias.shape[1], _stream()), "attention_chunked_mma", 2 if splits > 1 else 1)
+
+
 def swiglu_fusable(hidden: int, inter: int, dtype: torch.dtype) -> bool:
     """Whether gate and up can be one product whose epilogue applies silu(gate) * up: bfloat16,
     rows on 16-byte boundaries, and an intermediate size that is a multiple of 64 (the weights
@@ -1460,12 +1603,12 @@ def interleave_gate_up(gate: torch.Tensor, up: torch.Tensor) -> torch.Tensor:
     return torch.stack([gate.view(inter // 64, 64, k), up.view(inter // 64, 64, k)], dim=1).reshape(2 * inter, k).contiguous()
 
 
-def matmul_swiglu(a: torch.Tensor, w_gate_up: torch.Tensor, out: torch.Tensor) -> None:
-    """out[M, I] = silu(a @ gate^T) * (a @ up^T) in one kernel; ``w_gate_up`` from ``interleave_gate_up``."""
+def matmul_swiglu(a: torch.Tensor, w_gate_up: torch.Tensor, out: torch.Tensor, activation: str = "silu") -> None:
+    """out[M, I] = act(a @ gate^T) * (a @ up^T) in one kernel; ``w_gate_up`` from ``interleave_gate_up``."""
     if weights_as_rows(a.shape[0], w_gate_up.shape[0], swiglu=True):
-        gemm_skinny(a, w_gate_up, out, swiglu=True)
+        gemm_skinny(a, w_gate_up, out, swiglu=True, activation=activation)
     else:
-        gemm_tcgen05(a, w_gate_up, out, swiglu=True)
+        gemm_tcgen05(a, w_gate_up, out, swiglu=True, activation=activation)
 
 
 def attention_tcgen05(q: torch.Tensor, q_stride: int, out: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Tensor,

@@ -7,7 +7,9 @@
 // and the skip D) or one number per (token, head, row of S) (gated linear attention: c = 1, D = 0).  k and q may be
 // shared by the heads of a group (head h reads group h / (heads / groups)).  Everything inside the recurrence is
 // 32-bit; k, q and v are read in their own type (float32, or the compute dtype straight from a projection), q times
-// q_scale.
+// q_scale.  A normaliser (a matrix memory with exponential gates, mLSTM) is one more column of S that is fed by c k alone:
+//
+//   n_t = diag(a_t) n_(t-1) + c_t k_t;     den_t = max(|n_t . q_t|, floor_t) + den_eps           [rows, heads]
 //
 //   outer_recurrence_kernel<TI, NPT>   a CTA per (sequence, head, block of columns of S).  A column of S is cut over
 //       L lanes of one warp, lane l holding rows l, l + L, ... (NPT of them, in registers); tokens arrive in tiles
@@ -41,9 +43,17 @@ struct OuterArgs {
     int vec_state;                                   // every row piece of four columns of S is 16-byte aligned
     int vec_in;                                      // k, q and a can be read four elements at a time
     float q_scale;
+    float* norm_state;                               // the slot's n at norm_state + slot * ld_state, [heads, N], or null
+    const float* floor;                              // [rows, heads]
+    float* den;                                      // [rows, heads]
+    float den_eps;
 };
 
-template <typename TI, int NPT>
+__device__ __forceinline__ float or_den(const OuterArgs& A, size_t row, int h, float dot) {
+    return fmaxf(fabsf(dot), A.floor[row * A.heads + h]) + A.den_eps;
+}
+
+template <typename TI, int NPT, bool NORM>
 __global__ void __launch_bounds__(OR_THREADS, 1)
 outer_recurrence_kernel(const OuterArgs A) {
     pdl_launch_dependents();
@@ -68,6 +78,16 @@ outer_recurrence_kernel(const OuterArgs A) {
     for (int i = 0; i < NPT; ++i) {
         const int n = i * L + lane;
         S[i] = (live && n < N) ? S_slot[(size_t)n * P + col] : 0.f;
+    }
+    // the normaliser: the lanes of the first column of S carry it too
+    const bool has_norm = NORM && blockIdx.x == 0 && threadIdx.x < 32;
+    const bool in_norm = has_norm && threadIdx.x < L;
+    float* n_slot = NORM ? A.norm_state + (size_t)A.seq_slots[s] * A.ld_state + (size_t)h * N : nullptr;
+    float nS[NORM ? NPT : 1];
+#pragma unroll
+    for (int i = 0; i < (NORM ? NPT : 0); ++i) {
+        const int n = i * L + lane;
+        nS[i] = (in_norm && n < N) ? n_slot[n] : 0.f;
     }
     const TI* qp = (const TI*)A.q; const TI* kp = (const TI*)A.k; const TI* vp = (const TI*)A.v;
     const float skip = A.skip != nullptr ? A.skip[h] : 0.f;
@@ -131,7 +151,25 @@ outer_recurrence_kernel(const OuterArgs A) {
             }
             for (int o = L >> 1; o > 0; o >>= 1) acc += __shfl_xor_sync(0xffffffffu, acc, o);
             if (lane == 0 && live) A.y[(size_t)(row0 + t0 + tt) * A.ld_y + (size_t)h * P + col] = fmaf(skip, vv, acc);
+            if (NORM && has_norm) {
+                float dot = 0.f;
+#pragma unroll
+                for (int i = 0; i < (NORM ? NPT : 0); ++i) {
+                    const int n = i * L + lane;
+                    if (in_norm && n < N) {
+                        nS[i] = fmaf(A.a_per_row ? aa[n] : aa[0], nS[i], kk[n]);
+                        dot = fmaf(nS[i], qq[n], dot);
+                    }
+                }
+                for (int o = L >> 1; o > 0; o >>= 1) dot += __shfl_xor_sync(0xffffffffu, dot, o);
+                if (threadIdx.x == 0) A.den[(size_t)(row0 + t0 + tt) * A.heads + h] = or_den(A, (size_t)(row0 + t0 + tt), h, dot);
+            }
         }
+    }
+#pragma unroll
+    for (int i = 0; i < (NORM ? NPT : 0); ++i) {
+        const int n = i * L + lane;
+        if (in_norm && n < N) n_slot[n] = nS[i];
     }
 #pragma unroll
     for (int i = 0; i < NPT; ++i) {
@@ -154,7 +192,8 @@ __device__ __forceinline__ void or_ld4(const bf16* p, float (&x)[4]) {
 // k, q (and a) and C of v for 3 R C multiply-adds, and only the column sums cross lanes.  A warp holds LR = 32 / CGW lanes
 // along the rows (lane = column group + CGW * row group; row n = row group + LR * i), so neighbouring lanes hold
 // neighbouring columns of a row.  Rows from N to LR * R are zero in shared memory and change nothing.
-template <typename TI, int R, int C>
+// NORM: with the normaliser, which the warp of the CTA's first columns of S carries (every column group of it alike).
+template <typename TI, int R, int C, bool NORM>
 __global__ void __launch_bounds__(256)
 outer_recurrence_slab_kernel(const OuterArgs A) {
     pdl_launch_dependents();
@@ -187,6 +226,16 @@ outer_recurrence_slab_kernel(const OuterArgs A) {
             for (int j = 0; j < C; ++j) S[i][j] = (live && n < N) ? S_slot[(size_t)n * P + col0 + j] : 0.f;
         }
     }
+    const bool norm = NORM && blockIdx.x == 0 && warp == 0;
+    float* n_slot = NORM ? A.norm_state + (size_t)A.seq_slots[s] * A.ld_state + (size_t)h * N : nullptr;
+    float nS[NORM ? R : 1];
+    if constexpr (NORM) {
+#pragma unroll
+        for (int i = 0; i < R; ++i) {
+            const int n = rg + LR * i;
+            nS[i] = (norm && n < N) ? n_slot[n] : 0.f;
+        }
+    }
     const TI* qp = (const TI*)A.q; const TI* kp = (const TI*)A.k; const TI* vp = (const TI*)A.v;
     const float skip = A.skip != nullptr ? A.skip[h] : 0.f;
     // one tile's tokens: decay, update, multiply by q, add the lanes' column sums
@@ -217,6 +266,19 @@ outer_recurrence_slab_kernel(const OuterArgs A) {
                 float* y = A.y + (size_t)(row0 + t0 + tt) * A.ld_y + (size_t)h * P + col0;
 #pragma unroll
                 for (int j = 0; j < C; ++j) y[j] = fmaf(skip, v[j], acc[j]);
+            }
+            if constexpr (NORM) {
+                if (norm) {
+                    float dot = 0.f;
+#pragma unroll
+                    for (int i = 0; i < R; ++i) {
+                        const int n = rg + LR * i;
+                        nS[i] = fmaf(A.a_per_row ? aa[n] : a0, nS[i], kk[n]);
+                        dot = fmaf(nS[i], qq[n], dot);
+                    }
+                    for (int o = cgw; o < 32; o <<= 1) dot += __shfl_xor_sync(0xffffffffu, dot, o);
+                    if (lane == 0) A.den[(size_t)(row0 + t0 + tt) * A.heads + h] = or_den(A, (size_t)(row0 + t0 + tt), h, dot);
+                }
             }
         }
     };
@@ -268,6 +330,13 @@ outer_recurrence_slab_kernel(const OuterArgs A) {
             for (int tt = threadIdx.x; tt < nt; tt += threads) sm[tt * per_tok + 2 * Np] = A.a[(size_t)(row0 + t0 + tt) * A.ld_a + h];
         __syncthreads();
         compute(t0, nt);
+    }
+    if constexpr (NORM) {
+#pragma unroll
+        for (int i = 0; i < R; ++i) {
+            const int n = rg + LR * i;
+            if (norm && lane % cgw == 0 && n < N) n_slot[n] = nS[i];
+        }
     }
 #pragma unroll
     for (int i = 0; i < R; ++i) {
@@ -322,13 +391,16 @@ decay_lowrank_kernel(const T* __restrict__ r1, long long ld_r1, int col, int ran
 
 using namespace kl;
 
-// in_dtype: the type of q, k and v (KL_F32 or KL_BF16).  a_per_row != 0: a is [rows, heads * N].
+// in_dtype: the type of q, k and v (KL_F32 or KL_BF16).  a_per_row != 0: a is [rows, heads * N].  norm_state (null: no normaliser)
+// lies in the slot's state like `state`, ld_state apart; floor and den are float32 [rows, heads].
 KL_API int kl_outer_recurrence(const void* q, long long ld_q, int q_col, const void* k, long long ld_k, int k_col, const void* v,
                                long long ld_v, int v_col, const float* a, long long ld_a, int a_per_row, const float* c,
                                long long ld_c, const float* skip, float* state, long long ld_state, float* y, long long ld_y,
                                const int* cu_tokens, const int* seq_slots, int n_seqs, int max_new, int heads, int groups, int N, int P,
-                               float q_scale, int in_dtype, cudaStream_t stream) {
+                               float q_scale, float* norm_state, const float* floor, float* den, float den_eps, int in_dtype,
+                               cudaStream_t stream) {
     if (n_seqs <= 0) return KL_OK;
+    if (norm_state != nullptr && (floor == nullptr || den == nullptr)) return KL_ERR_BAD_SIZE;
     if (heads <= 0 || groups <= 0 || heads % groups || N <= 0 || P <= 0 || N > 1024) return KL_ERR_BAD_SIZE;
     if (in_dtype != KL_F32 && in_dtype != KL_BF16) return KL_ERR_BAD_DTYPE;
     int sms = 0, dev = 0;
@@ -339,6 +411,7 @@ KL_API int kl_outer_recurrence(const void* q, long long ld_q, int q_col, const v
     A.a = a; A.ld_a = ld_a; A.c = c; A.ld_c = ld_c; A.skip = skip; A.state = state; A.ld_state = ld_state; A.y = y; A.ld_y = ld_y;
     A.cu_tokens = cu_tokens; A.seq_slots = seq_slots; A.heads = heads; A.groups = groups; A.N = N; A.P = P;
     A.a_per_row = a_per_row ? 1 : 0; A.q_scale = q_scale;
+    A.norm_state = norm_state; A.floor = floor; A.den = den; A.den_eps = den_eps;
     A.vec_state = ((uintptr_t)state % 16 == 0 && ld_state % 4 == 0 && P % 4 == 0) ? 1 : 0;
     {   // slabs of R x C in registers: the largest slab that still gives every SM eight warps, else the smallest that fits
         const int slabs[3][2] = {{8, 4}, {4, 4}, {2, 2}};
@@ -370,18 +443,23 @@ KL_API int kl_outer_recurrence(const void* q, long long ld_q, int q_col, const v
             A.vec_in = (N % 4 == 0 && (LR * R) % 4 == 0 && per_tok % 4 == 0 && quad(q, ld_q, q_col) && quad(k, ld_k, k_col) &&
                         (!a_per_row || ((uintptr_t)a % 16 == 0 && ld_a % 4 == 0))) ? 1 : 0;
             if (smem <= 200 * 1024) {
-#define KL_SLAB(TI, R_, C_)                                                                                          \
+#define KL_SLAB(TI, R_, C_, NM)                                                                                      \
     do {                                                                                                            \
         if (smem > 48 * 1024)                                                                                       \
-            KL_CUDA(cudaFuncSetAttribute(outer_recurrence_slab_kernel<TI, R_, C_>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem)); \
-        launch_kernel(outer_recurrence_slab_kernel<TI, R_, C_>, grid, threads, smem, stream, A);                    \
+            KL_CUDA(cudaFuncSetAttribute(outer_recurrence_slab_kernel<TI, R_, C_, NM>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem)); \
+        launch_kernel(outer_recurrence_slab_kernel<TI, R_, C_, NM>, grid, threads, smem, stream, A);                \
+    } while (0)
+#define KL_SLAB_N(TI, R_, C_)                                                                                       \
+    do {                                                                                                            \
+        if (norm_state != nullptr) KL_SLAB(TI, R_, C_, true); else KL_SLAB(TI, R_, C_, false);                      \
     } while (0)
 #define KL_SLAB_BY(TI)                                                                                              \
     do {                                                                                                            \
-        if (R == 8) KL_SLAB(TI, 8, 4); else if (R == 4) KL_SLAB(TI, 4, 4); else KL_SLAB(TI, 2, 2);                  \
+        if (R == 8) KL_SLAB_N(TI, 8, 4); else if (R == 4) KL_SLAB_N(TI, 4, 4); else KL_SLAB_N(TI, 2, 2);            \
     } while (0)
                 if (in_dtype == KL_F32) KL_SLAB_BY(float); else KL_SLAB_BY(bf16);
 #undef KL_SLAB_BY
+#undef KL_SLAB_N
 #undef KL_SLAB
                 KL_LAUNCH_CHECK();
                 return KL_OK;
@@ -405,11 +483,15 @@ KL_API int kl_outer_recurrence(const void* q, long long ld_q, int q_col, const v
     dim3 grid((P + cols - 1) / cols, heads, n_seqs);
     const size_t smem = (size_t)OR_TILE * (2 * N + (a_per_row ? N : 1) + cols) * sizeof(float);
     if (smem > 200 * 1024) return KL_ERR_BAD_SIZE;
-#define KL_OR(TI, NPT)                                                                                              \
+#define KL_OR_N(TI, NPT, NM)                                                                                        \
     do {                                                                                                            \
         if (smem > 48 * 1024)                                                                                       \
-            KL_CUDA(cudaFuncSetAttribute(outer_recurrence_kernel<TI, NPT>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem)); \
-        launch_kernel(outer_recurrence_kernel<TI, NPT>, grid, threads, smem, stream, A);                         \
+            KL_CUDA(cudaFuncSetAttribute(outer_recurrence_kernel<TI, NPT, NM>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem)); \
+        launch_kernel(outer_recurrence_kernel<TI, NPT, NM>, grid, threads, smem, stream, A);                        \
+    } while (0)
+#define KL_OR(TI, NPT)                                                                                              \
+    do {                                                                                                            \
+        if (norm_state != nullptr) KL_OR_N(TI, NPT, true); else KL_OR_N(TI, NPT, false);                            \
     } while (0)
 #define KL_OR_BY_NPT(TI)                                                                                            \
     do {                                                                                                            \
@@ -418,6 +500,7 @@ KL_API int kl_outer_recurrence(const void* q, long long ld_q, int q_col, const v
     if (in_dtype == KL_F32) KL_OR_BY_NPT(float); else KL_OR_BY_NPT(bf16);
 #undef KL_OR_BY_NPT
 #undef KL_OR
+#undef KL_OR_N
     KL_LAUNCH_CHECK();
     return KL_OK;
 }

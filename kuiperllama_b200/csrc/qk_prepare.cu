@@ -222,9 +222,154 @@ qk_prepare_vec_kernel(bf16* __restrict__ proj, long long ld, int q_col, int k_co
     }
 }
 
+// The preparation for attention whose q and k are normed over the WHOLE projection (all heads at once) and whose values
+// may be mixed with those of another layer; no rotation.  A CTA per (token, role):
+//
+//   role 0   q / sqrt(mean(q^2) + eps) * q_w  -> q_out
+//   role 1   k likewise                       -> the token's row of the key cache
+//   role 2   v, or (1 - lambda) v + lambda v_first -> the value cache; v as projected also -> v_keep where one is given
+//
+// The projections are rows in the compute dtype or float32 pieces [n_pieces][rows][ld] of a product whose K range was cut
+// (added in ascending order).  V: elements an access (8 where rows, heads and pointers allow 16-byte accesses, else 1).
+struct RowPrepare {
+    const void* rows; const float* pieces; int n_pieces; long long piece_stride; long long ld;
+    int q_col, k_col, v_col;
+    const float* q_w; const float* k_w; float eps; int norm;
+    void* q_out; long long q_ld;
+    void* k_cache; void* v_cache; const int* block_table; int blocks_per_seq;
+    const void* v_first; long long v_first_ld; const float* lambda; void* v_keep;
+    const int* positions; const int* token_slot;
+    int H, KV, hd, vd;
+};
+template <typename T, int V>
+__device__ __forceinline__ void rp_load(const RowPrepare& A, size_t at, float (&x)[V]) {
+    if (A.pieces != nullptr) {
+#pragma unroll
+        for (int e = 0; e < V; ++e) x[e] = 0.f;
+        for (int z = 0; z < A.n_pieces; ++z) {
+            const float* p = A.pieces + (size_t)z * A.piece_stride + at;
+            if constexpr (V == 8) {
+                const float4 a = *reinterpret_cast<const float4*>(p), b = *reinterpret_cast<const float4*>(p + 4);
+                x[0] += a.x; x[1] += a.y; x[2] += a.z; x[3] += a.w; x[4] += b.x; x[5] += b.y; x[6] += b.z; x[7] += b.w;
+            } else x[0] += p[0];
+        }
+        return;
+    }
+    const T* p = (const T*)A.rows + at;
+    if constexpr (V == 8 && sizeof(T) == 2) {
+        const uint4 raw = *reinterpret_cast<const uint4*>(p);
+        const __nv_bfloat162* b = reinterpret_cast<const __nv_bfloat162*>(&raw);
+#pragma unroll
+        for (int e = 0; e < 4; ++e) { const float2 f = __bfloat1622float2(b[e]); x[2 * e] = f.x; x[2 * e + 1] = f.y; }
+    } else {
+#pragma unroll
+        for (int e = 0; e < V; ++e) x[e] = to_f32(p[e]);
+    }
+}
+template <typename T, int V>
+__device__ __forceinline__ void rp_store(T* p, const float (&x)[V]) {
+    if constexpr (V == 8 && sizeof(T) == 2) {
+        uint4 out;
+        __nv_bfloat162* o = reinterpret_cast<__nv_bfloat162*>(&out);
+#pragma unroll
+        for (int e = 0; e < 4; ++e) o[e] = __floats2bfloat162_rn(x[2 * e], x[2 * e + 1]);
+        *reinterpret_cast<uint4*>(p) = out;
+    } else {
+#pragma unroll
+        for (int e = 0; e < V; ++e) p[e] = from_f32<T>(x[e]);
+    }
+}
+template <typename T, int V>
+__global__ void __launch_bounds__(256)
+qk_row_prepare_kernel(const RowPrepare A) {
+    pdl_launch_dependents();
+    pdl_wait();
+    extern __shared__ __align__(16) float smem[];       // [width]: a thread reads back its own elements only
+    __shared__ float scratch[33];
+    const int t = blockIdx.x, role = blockIdx.y;
+    const int slot = A.token_slot[t];
+    if (slot < 0) return;                               // a padding row
+    const int pos = A.positions[t];
+    if (role > 0 && A.k_cache == nullptr && !(role == 2 && A.v_keep != nullptr)) return;
+    const int width = role == 0 ? A.H * A.hd : (role == 1 ? A.KV * A.hd : A.KV * A.vd);
+    const size_t at = (size_t)t * A.ld + (role == 0 ? A.q_col : (role == 1 ? A.k_col : A.v_col));
+    if (role == 2) {
+        const float lam = A.v_first != nullptr ? A.lambda[0] : 0.f;
+        for (int i = threadIdx.x * V; i < width; i += blockDim.x * V) {
+            float x[V];
+            rp_load<T, V>(A, at + i, x);
+            if (A.v_keep != nullptr) rp_store<T, V>((T*)A.v_keep + (size_t)t * width + i, x);
+            if (A.k_cache == nullptr) continue;
+            if (A.v_first != nullptr) {
+                const T* f = (const T*)A.v_first + (size_t)t * A.v_first_ld + i;
+#pragma unroll
+                for (int e = 0; e < V; ++e) x[e] = (1.0f - lam) * x[e] + lam * to_f32(f[e]);
+            }
+            const int g = i / A.vd, e0 = i - g * A.vd;
+            rp_store<T, V>((T*)A.v_cache + cache_row_offset(A.block_table, A.blocks_per_seq, slot, pos, g, A.KV, A.vd) + e0, x);
+        }
+        return;
+    }
+    float ss = 0.f;
+    for (int i = threadIdx.x * V; i < width; i += blockDim.x * V) {
+        float x[V];
+        rp_load<T, V>(A, at + i, x);
+#pragma unroll
+        for (int e = 0; e < V; ++e) { ss += x[e] * x[e]; smem[i + e] = x[e]; }
+    }
+    float inv = 1.f;
+    if (A.norm) inv = 1.0f / sqrtf(block_sum(ss, scratch) / (float)width + A.eps);
+    const float* w = role == 0 ? A.q_w : A.k_w;
+    for (int i = threadIdx.x * V; i < width; i += blockDim.x * V) {
+        float x[V];
+#pragma unroll
+        for (int e = 0; e < V; ++e) x[e] = smem[i + e] * inv * (w != nullptr ? w[i + e] : 1.f);
+        if (role == 0) {
+            rp_store<T, V>((T*)A.q_out + (size_t)t * A.q_ld + i, x);
+        } else {
+            const int g = i / A.hd, e0 = i - g * A.hd;
+            rp_store<T, V>((T*)A.k_cache + cache_row_offset(A.block_table, A.blocks_per_seq, slot, pos, g, A.KV, A.hd) + e0, x);
+        }
+    }
+}
+
 }  // namespace kl
 
 using namespace kl;
+
+// rows (compute dtype, `ld` elements apart; q_out may be their q columns) or pieces (float32 [n_pieces][..][ld], piece_stride
+// elements apart): q heads from column q_col, k heads from k_col, v heads from v_col.  v_first (compute dtype) with lambda
+// (float32, one number on the device) or null; v_keep [n_tokens, KV * vd] or null; caches both null: q (and v_keep) alone.
+KL_API int kl_qk_row_prepare(const void* rows, const float* pieces, int n_pieces, long long piece_stride, long long ld, int q_col,
+                             int k_col, int v_col, int norm, float eps, const float* q_w, const float* k_w, void* q_out,
+                             long long q_ld, void* k_cache, void* v_cache, const int* block_table, int blocks_per_seq,
+                             const void* v_first, long long v_first_ld, const float* lambda, void* v_keep, const int* positions,
+                             const int* token_slot, int n_tokens, int H, int KV, int hd, int vd, int dtype, cudaStream_t stream) {
+    if (n_tokens <= 0) return KL_OK;
+    if (H <= 0 || KV <= 0 || hd <= 0 || vd <= 0 || (rows == nullptr) == (pieces == nullptr) || (pieces != nullptr && n_pieces < 1)) return KL_ERR_BAD_SIZE;
+    if ((k_cache == nullptr) != (v_cache == nullptr) || (v_first != nullptr && lambda == nullptr) || q_out == nullptr) return KL_ERR_BAD_SIZE;
+    if (dtype != KL_F32 && dtype != KL_BF16) return KL_ERR_BAD_DTYPE;
+    RowPrepare A{rows, pieces, n_pieces, piece_stride, ld, q_col, k_col, v_col, q_w, k_w, eps, norm, q_out, q_ld, k_cache, v_cache,
+                 block_table, blocks_per_seq, v_first, v_first_ld, lambda, v_keep, positions, token_slot, H, KV, hd, vd};
+    const size_t smem = (size_t)(H > KV ? H : KV) * hd * sizeof(float);
+    if (smem > 200 * 1024) return KL_ERR_BAD_SIZE;
+    const uintptr_t ptrs = (uintptr_t)rows | (uintptr_t)pieces | (uintptr_t)q_out | (uintptr_t)k_cache | (uintptr_t)v_cache | (uintptr_t)v_first |
+                           (uintptr_t)v_keep;
+    const bool wide = dtype == KL_BF16 && hd % 8 == 0 && vd % 8 == 0 && ld % 8 == 0 && q_ld % 8 == 0 && v_first_ld % 8 == 0 && q_col % 8 == 0 &&
+                      k_col % 8 == 0 && v_col % 8 == 0 && piece_stride % 8 == 0 && (ptrs & 15) == 0;
+    const dim3 grid(n_tokens, 3);
+#define KL_RP(T, V)                                                                                                                \
+    do {                                                                                                                           \
+        if (smem > 40 * 1024) KL_CUDA(cudaFuncSetAttribute(qk_row_prepare_kernel<T, V>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem)); \
+        launch_kernel(qk_row_prepare_kernel<T, V>, grid, 256, smem, stream, A);                                                    \
+    } while (0)
+    if (dtype == KL_F32) KL_RP(float, 1);
+    else if (wide) KL_RP(bf16, 8);
+    else KL_RP(bf16, 1);
+#undef KL_RP
+    KL_LAUNCH_CHECK();
+    return KL_OK;
+}
 
 // proj: rows of `ld` elements; q heads from column q_col, k heads from k_col, v heads from v_col (< 0: none).
 // Caches: [pages, KV, PAGE, hd] and [pages, KV, PAGE, vd]; both null: a layer that only reads a cache.

@@ -13,10 +13,13 @@ namespace kl {
 
 // out[t, :] = scale * table[ids[t], :] as float32 (scale 1 for a plain gather).  An id outside
 // [0, vocab) writes zeros and sets *error_flag (KuiperLLama skips such a row silently,
-// emb_kernel.cu:11-13).
+// emb_kernel.cu:11-13).  With `freq` (float32 [2, ceil(hidden / 2)]: every pair's frequency and what its rounding to float32
+// left over) a sinusoid of the token's position is added: entry 2i gets sin(p f_i), entry 2i + 1 cos(p f_i).  The angle
+// is a 32-bit product; its rounding error and the frequency's (1e-4 at position 2,000) come in as a first-order correction.
 template <typename T>
 __global__ void embedding_kernel(const int* __restrict__ ids, const T* __restrict__ table, float* __restrict__ out,
-                                 int hidden, int vocab, float scale, int* __restrict__ error_flag) {
+                                 int hidden, int vocab, float scale, const int* __restrict__ positions, const float* __restrict__ freq,
+                                 int* __restrict__ error_flag) {
     pdl_launch_dependents();
     pdl_wait();
     const int t = blockIdx.x;
@@ -28,6 +31,19 @@ __global__ void embedding_kernel(const int* __restrict__ ids, const T* __restric
         return;
     }
     const T* row = table + (size_t)id * hidden;
+    if (freq != nullptr) {
+        const int pairs = (hidden + 1) / 2;
+        const float p = (float)positions[t];
+        for (int i = threadIdx.x; i < pairs; i += blockDim.x) {
+            const float angle = p * freq[i];
+            const float rest = fmaf(p, freq[i], -angle) + p * freq[pairs + i];
+            float sn, cs;
+            sincosf(angle, &sn, &cs);
+            o[2 * i] = fmaf(scale, to_f32(row[2 * i]), fmaf(rest, cs, sn));
+            if (2 * i + 1 < hidden) o[2 * i + 1] = fmaf(scale, to_f32(row[2 * i + 1]), fmaf(-rest, sn, cs));
+        }
+        return;
+    }
     for (int i = threadIdx.x; i < hidden; i += blockDim.x) o[i] = scale * to_f32(row[i]);
 }
 
@@ -168,9 +184,10 @@ add_rmsnorm_kernel(float* __restrict__ residual, const T* __restrict__ delta, co
     }
 }
 
-// out[t, i] = silu(gu[t, i]) * gu[t, inter + i]; gu is [tokens, 2 * inter] (gate columns first).
+// out[t, i] = act(gu[t, i]) * gu[t, inter + i]; gu is [tokens, 2 * inter] (gate columns first); act = silu, or with
+// gelu the tanh form of gelu.
 template <typename T>
-__global__ void swiglu_kernel(const T* __restrict__ gu, T* __restrict__ out, int tokens, int inter) {
+__global__ void swiglu_kernel(const T* __restrict__ gu, T* __restrict__ out, int tokens, int inter, int gelu) {
     pdl_launch_dependents();
     pdl_wait();
     const size_t n = (size_t)tokens * inter;
@@ -179,7 +196,8 @@ __global__ void swiglu_kernel(const T* __restrict__ gu, T* __restrict__ out, int
         const int i = (int)(idx - t * inter);
         const float g = to_f32(gu[t * 2 * inter + i]);
         const float u = to_f32(gu[t * 2 * inter + inter + i]);
-        out[idx] = from_f32<T>(g * (1.0f / (1.0f + expf(-g))) * u);
+        const float a = gelu ? 0.5f * g * (1.0f + tanhf(0.7978845608028654f * (g + 0.044715f * g * g * g))) : g * (1.0f / (1.0f + expf(-g)));
+        out[idx] = from_f32<T>(a * u);
     }
 }
 
@@ -212,13 +230,14 @@ KL_API int kl_logit_transform(float* logits, long long ld, int rows, int vocab, 
 }
 
 KL_API int kl_embedding(const int* ids, int n_tokens, const void* table, int table_dtype, int vocab, int hidden,
-                        float scale, float* out, int* error_flag, cudaStream_t stream) {
+                        float scale, const int* positions, const float* freq, float* out, int* error_flag, cudaStream_t stream) {
     if (n_tokens <= 0) return KL_OK;
+    if (freq != nullptr && positions == nullptr) return KL_ERR_BAD_SIZE;
     const int threads = hidden >= 1024 ? 256 : 128;
     if (table_dtype == KL_F32)
-        launch_kernel(embedding_kernel<float>, n_tokens, threads, 0, stream, ids, (const float*)table, out, hidden, vocab, scale, error_flag);
+        launch_kernel(embedding_kernel<float>, n_tokens, threads, 0, stream, ids, (const float*)table, out, hidden, vocab, scale, positions, freq, error_flag);
     else if (table_dtype == KL_BF16)
-        launch_kernel(embedding_kernel<bf16>, n_tokens, threads, 0, stream, ids, (const bf16*)table, out, hidden, vocab, scale, error_flag);
+        launch_kernel(embedding_kernel<bf16>, n_tokens, threads, 0, stream, ids, (const bf16*)table, out, hidden, vocab, scale, positions, freq, error_flag);
     else
         return KL_ERR_BAD_DTYPE;
     KL_LAUNCH_CHECK();
@@ -247,15 +266,15 @@ KL_API int kl_add_rmsnorm(float* residual, const void* delta, const float* parti
     return KL_OK;
 }
 
-KL_API int kl_swiglu(const void* gate_up, void* out, int tokens, int inter, int dtype, cudaStream_t stream) {
+KL_API int kl_swiglu(const void* gate_up, void* out, int tokens, int inter, int gelu, int dtype, cudaStream_t stream) {
     if (tokens <= 0) return KL_OK;
     const size_t n = (size_t)tokens * inter;
     const int threads = 256;
     const int blocks = kl::strided_grid(n, threads, 16);
     if (dtype == KL_F32)
-        launch_kernel(swiglu_kernel<float>, blocks, threads, 0, stream, (const float*)gate_up, (float*)out, tokens, inter);
+        launch_kernel(swiglu_kernel<float>, blocks, threads, 0, stream, (const float*)gate_up, (float*)out, tokens, inter, gelu);
     else if (dtype == KL_BF16)
-        launch_kernel(swiglu_kernel<bf16>, blocks, threads, 0, stream, (const bf16*)gate_up, (bf16*)out, tokens, inter);
+        launch_kernel(swiglu_kernel<bf16>, blocks, threads, 0, stream, (const bf16*)gate_up, (bf16*)out, tokens, inter, gelu);
     else
         return KL_ERR_BAD_DTYPE;
     KL_LAUNCH_CHECK();

@@ -106,12 +106,14 @@ class DecoderModel:
         """Run embedding and all scheduled layers: the float32 residual stream and the last
         feed-forward's output that is still to be added to it."""
         step.allow_stream_fusion = self.stream_fusion and step.is_decode
+        step.shared.clear()
         residual = torch.empty((step.n_tokens, self.spec.hidden_size), dtype=torch.float32, device=self.runtime.device)
+        position = getattr(self.blocks[self.spec.schedule[0].layer], "position", None)
         ops.embedding(step.token_ids[:step.n_tokens], self.embedding, residual, self.error_flag,
-                      scale=1.0 if self.spec.embedding_multiplier is None else float(self.spec.embedding_multiplier))
-        first = self.blocks[self.spec.schedule[0].layer]
-        if getattr(first, "position", None) is not None:
-            first.position.add_to_embeddings(residual, step)
+                      scale=1.0 if self.spec.embedding_multiplier is None else float(self.spec.embedding_multiplier),
+                      positions=step.positions, freq=position.embedding_frequencies() if position is not None else None)
+        if position is not None:
+            position.add_to_embeddings(residual, step)
         pending = None
         schedule = self.spec.schedule
         for i, entry in enumerate(schedule):

@@ -13,7 +13,7 @@ counts partly compiled in.
 """
 from __future__ import annotations
 
-from dataclasses import dataclass
+from dataclasses import dataclass, field
 from typing import Callable, Dict, List, Optional
 
 import torch
@@ -66,6 +66,9 @@ class StepContext:
     # the residual stream into the products at all.
     next_norm: Optional["Norm"] = None
     allow_stream_fusion: bool = False
+    # What a layer leaves for later layers of the same step, by a name the parts agree on (the values that later layers mix
+    # into theirs, for instance).  It starts empty with every step.
+    shared: Dict[str, torch.Tensor] = field(default_factory=dict)
 
 
 @dataclass
@@ -169,9 +172,14 @@ class Norm(Part):
 class PositionEncoding(Part):
     """A position encoding either rotates queries and keys inside the mixer (``rotary()``
     returns the inverse frequencies and the rotated width) or changes the embeddings before
-    the first layer (``add_to_embeddings``), or both."""
+    the first layer (``add_to_embeddings``), or both.  One that adds a sinusoid to the embeddings gives its
+    frequencies (``embedding_frequencies``, float32 [2, ceil(hidden / 2)]: every pair's frequency and what its rounding left
+    over), and the embedding kernel adds it itself."""
 
     def rotary(self) -> Optional[tuple]:
+        return None
+
+    def embedding_frequencies(self) -> Optional[torch.Tensor]:
         return None
 
     def add_to_embeddings(self, residual: torch.Tensor, step: StepContext) -> None:

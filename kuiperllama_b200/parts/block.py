@@ -103,6 +103,8 @@ class ParallelBlock:
 
         x += (mixer(norm1(x)) + feed_forward(norm2(x)))          (x += mixer(norm1(x)) without a feed-forward)
 
+    Without a feed-forward norm both sublayers read the one norm's rows, h = norm1(x): x += mixer(h) + feed_forward(h).
+
     The two RMS norms share their root mean square, so one kernel adds what the block before left
     pending (32-bit), writes the stream and makes both normalised rows; the block's own two results
     travel on as ``DeltaSum`` to the norm that reads the stream next.  Norms of other kinds run one
@@ -115,7 +117,7 @@ class ParallelBlock:
 
     def forward(self, residual: torch.Tensor, pending, step: StepContext, cache: CacheView):
         step.residual_sink = None
-        a, b = self.mixer_norm, self.feed_forward_norm if self.feed_forward is not None else None
+        a, b = self.mixer_norm, self.feed_forward_norm if self.feed_forward is not None else None      # b None: one norm for both
         if b is not None and hasattr(a, "forward_pair") and type(a) is type(b) and a.eps == b.eps:
             h1, h2 = a.forward_pair(residual, pending, b)
         else:
@@ -123,6 +125,8 @@ class ParallelBlock:
             if isinstance(h1, NormedLazy):
                 h1 = h1.dense()
             h2 = b.forward(residual, None, step.n_tokens) if b is not None else None
+        if h2 is None:
+            h2 = h1
         mixed = self.mixer.forward(h1, step, cache)
         if self.feed_forward is None:
             return residual, mixed

@@ -74,6 +74,7 @@ class StackedInput:
         self.linear: Optional[Linear] = None
         self.total = 0
         self.last: Optional[torch.Tensor] = None     # the product of the latest forward, [m, total]
+        self.rows: Optional[torch.Tensor] = None     # and the rows it read
 
     def add(self, name: str, weight: torch.Tensor) -> None:
         if self.linear is not None:
@@ -96,12 +97,15 @@ class StackedInput:
     def column(self, name: str) -> int:
         return self.columns[name][0]
 
-    def forward(self, x: torch.Tensor) -> torch.Tensor:
+    def forward(self, x: torch.Tensor, allow_partials: bool = False) -> torch.Tensor:
+        """[m, total].  With ``allow_partials`` the result may be float32 pieces [S, m, total] (see ``Linear.forward``), which the
+        caller's kernel adds; ``view`` is then not to be used."""
         if self.linear is None:
             self._pad()
             self.linear = Linear(torch.cat([w for _, w in self._pieces], dim=0), self.runtime)
             self._pieces = []
-        self.last = self.linear.forward(x)
+        self.rows = x
+        self.last = self.linear.forward(x, allow_partials=allow_partials)
         return self.last
 
     def view(self, name: str) -> torch.Tensor:

@@ -1,4 +1,5 @@
-"""Recurrent mixers whose state is a matrix per head, fed by outer products: a state-space layer and gated linear attention."""
+"""Recurrent mixers whose state is a matrix per head, fed by outer products: a state-space layer, gated linear attention and a
+matrix memory with exponential gates."""
 from __future__ import annotations
 
 from typing import Dict, Optional
@@ -147,3 +148,71 @@ class GatedLinearAttentionMixer(BranchMixer):
         ops.outer_recurrence(stacked.view(tag + "q"), stacked.view(tag + "k"), stacked.view(tag + "v"), alpha, cache.state, o, step,
                              self.H, self.H, self.d, self.dv, q_scale=self.q_scale)
         ops.head_rmsnorm_gate(o, stacked.view(tag + "g"), self.norm_weight, out, self.H, self.dv, self.norm_eps, out_scale=out_scale)
+
+
+@register_mixer("mlstm")
+class MLSTMMixer(BranchMixer):
+    """The matrix memory with exponential gates of Beck et al., "xLSTM: Extended Long Short-Term Memory" (2024), in its recurrent
+    form.  q = Wq n * q_scale and k = Wk n (heads x dim), v = Wv n (heads x vdim).  Per head, with soft(z) = cap tanh(z / cap), a
+    log input gate i = soft(Wi n + bi) and a log forget gate f = logsigmoid(soft(Wf n + bf)); S [dim, vdim], z [dim] and m
+    start at zero:
+
+        m_t = max(f_t + m_(t-1), i_t)
+        S_t = exp(f_t + m_(t-1) - m_t) S_(t-1) + exp(i_t - m_t) k_t v_t^T;      z_t likewise with k_t alone
+        o_t = S_t^T q_t / (max(|z_t . q_t|, exp(-m_t)) + den_eps)
+
+    then each head's o over its root mean square (over vdim) times a weight per channel, times sigmoid(Wg n), and the
+    output projection.  The gates' projections, the gates, the maximum, S, z, o and the norm are 32-bit; the slot's state is S as
+    [heads, dim, vdim], z as [heads, dim] and m as [heads], float32.  Spec: ``hidden_size``, ``heads``, ``dim``, ``vdim``, ``cap``,
+    ``q_scale``, ``den_eps``, ``norm_eps`` and ``names`` (q, k, v, g, o, norm, i, i_bias, f, f_bias).  KuiperLLama has no
+    recurrent mixer (its mixer is mha_kernel.cu:61,74-106)."""
+
+    @classmethod
+    def manifest(cls, spec: PartSpec, prefix: str) -> Dict[str, TensorDecl]:
+        hid, H, d, dv, n = (spec[k] for k in ("hidden_size", "heads", "dim", "vdim", "names"))
+        return {prefix + n["q"]: TensorDecl((H * d, hid)), prefix + n["k"]: TensorDecl((H * d, hid)),
+                prefix + n["v"]: TensorDecl((H * dv, hid)), prefix + n["g"]: TensorDecl((H * dv, hid)),
+                prefix + n["o"]: TensorDecl((hid, H * dv)), prefix + n["norm"]: TensorDecl((H * dv,), role="vector", init="one_plus_normal"),
+                prefix + n["i"]: TensorDecl((H, hid)), prefix + n["i_bias"]: TensorDecl((H,), role="vector"),
+                prefix + n["f"]: TensorDecl((H, hid)), prefix + n["f_bias"]: TensorDecl((H,), role="vector")}
+
+    def __init__(self, spec, prefix, tensors, runtime: Runtime, position: Optional[PositionEncoding] = None):
+        super().__init__(spec, prefix, tensors, runtime, position)
+        self.hidden = int(spec["hidden_size"])
+        self.H, self.d, self.dv = (int(spec[k]) for k in ("heads", "dim", "vdim"))
+        self.cap, self.q_scale = float(spec["cap"]), float(spec["q_scale"])
+        self.den_eps, self.norm_eps = float(spec["den_eps"]), float(spec["norm_eps"])
+        if not self.cap > 0:
+            raise ValueError(f"the gates' cap must be positive, got {self.cap}")
+        if self.d > 1024:
+            raise ValueError(f"a key size of {self.d} is above the recurrence kernel's 1,024")
+        n = spec["names"]
+        self._w = {k: tensors[prefix + n[k]] for k in ("q", "k", "v", "g")}
+        self.o_weight = tensors[prefix + n["o"]]
+        self.core_width = self.H * self.dv
+        f32 = lambda name: tensors[prefix + name].to(device=runtime.device, dtype=torch.float32).contiguous()
+        self.gate_weight = torch.cat([tensors[prefix + n[k]].to(device=runtime.device, dtype=runtime.dtype) for k in ("i", "f")]).contiguous()
+        self.gate_bias = torch.cat([f32(n["i_bias"]), f32(n["f_bias"])]).contiguous()
+        self.norm_weight = f32(n["norm"])
+        self.z_off = self.H * self.d * self.dv
+        self.m_off = self.z_off + self.H * self.d
+
+    def state_request(self) -> Optional[StateRequest]:
+        return StateRequest((-(-(self.m_off + self.H) // 4) * 4,), torch.float32)       # a multiple of four: rows of S stay on 16-byte boundaries
+
+    def add_inputs(self, stacked: StackedInput, tag: str) -> None:
+        for k in ("q", "k", "v", "g"):
+            stacked.add(tag + k, self._w[k])
+        self._w = None
+
+    def core(self, stacked: StackedInput, tag: str, step: StepContext, cache: CacheView, out: torch.Tensor, out_scale: float) -> None:
+        n, dev = step.n_tokens, out.device
+        a, c, floor = ops.mlstm_gates(stacked.rows, self.gate_weight, self.gate_bias, self.cap, cache.state[:, self.m_off:], step)
+        make = torch.empty if n == step.n_seqs else torch.zeros
+        o = make((n, self.H * self.dv), dtype=torch.float32, device=dev)
+        den = (torch.empty if n == step.n_seqs else torch.ones)((n, self.H), dtype=torch.float32, device=dev)
+        ops.outer_recurrence(stacked.view(tag + "q"), stacked.view(tag + "k"), stacked.view(tag + "v"), a, cache.state, o, step,
+                             self.H, self.H, self.d, self.dv, c=c, q_scale=self.q_scale,
+                             normaliser=(cache.state[:, self.z_off:], floor, den, self.den_eps))
+        ops.head_rmsnorm_gate(o, stacked.view(tag + "g"), self.norm_weight, out, self.H, self.dv, self.norm_eps, out_scale=out_scale,
+                              divisor=den, gate_act="sigmoid")

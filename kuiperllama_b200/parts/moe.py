@@ -11,6 +11,7 @@ from ..csrc import ops
 from ..weights.loader import TensorDecl
 from .base import FeedForward, NormedLazy, Runtime, StepContext, register_feed_forward
 from .linear import Linear
+from .swiglu import SwiGLUFeedForward
 
 
 @register_feed_forward("moe")
@@ -25,11 +26,13 @@ class MoEFeedForward(FeedForward):
     With ``gated`` False an expert has no gate: f_e = W_down[e] act(W_up[e] n) with ``activation`` one of the element-wise
     activations (``ops.ACTIVATIONS``).  ``names['router_bias']``: a bias per expert joins the router's logits (32 bits).  With
     ``renormalise`` and no ``renorm_eps`` the weights are the softmax over the chosen logits alone.  ``shared_size``: one more
-    expert of that size and of the ungated form (``names['shared_up']``, ``names['shared_down']``) runs for every token and is
-    added, as a second float32 piece.
+    expert of that size and of the same form (``names['shared_up']``, ``names['shared_down']``, gated also
+    ``names['shared_gate']``) runs for every token and is added, as a second float32 piece.  ``scores`` "sigmoid": s = sigmoid(z),
+    each expert by itself; ``names['correction']``: a number per expert that joins the scores for the choice (of groups
+    too) but not for the weights; ``router_scale`` multiplies the weights.
 
     With ``groups`` > 1 the experts form that many equal groups of neighbours; a group's score is the largest score in
-    it, and only experts of the ``keep_groups`` best groups can be chosen.
+    it (or the sum of its ``group_top`` largest), and only experts of the ``keep_groups`` best groups can be chosen.
 
     Routing stays on the device (``ops.moe_route`` / ``moe_plan``): the (token, choice) pairs are sorted by
     expert into a list padded to whole tiles, one grouped product makes gate, up and the activation for
@@ -40,7 +43,8 @@ class MoEFeedForward(FeedForward):
     otherwise (float32, odd sizes).
 
     Spec: ``hidden_size``, ``experts``, ``top``, ``expert_size``, ``limit``, ``alpha``, ``shift``, ``renormalise``,
-    ``renorm_eps``, ``groups``, ``keep_groups``, ``gated``, ``activation``, ``shared_size``, ``names``: router and, with ``{e}`` for the
+    ``renorm_eps``, ``groups``, ``keep_groups``, ``group_top``, ``scores``, ``router_scale``, ``gated``, ``activation``,
+    ``shared_size``, ``names``: router and, with ``{e}`` for the
     expert's number, gate, up, down.  KuiperLLama's only feed-forward is
     the dense SwiGLU (kuiper/source/model/llama3.cpp:692-718)."""
 
@@ -56,12 +60,16 @@ class MoEFeedForward(FeedForward):
         m = {prefix + n["router"]: TensorDecl((E, hid))}
         if n.get("router_bias"):
             m[prefix + n["router_bias"]] = TensorDecl((E,), role="vector")
+        if n.get("correction"):
+            m[prefix + n["correction"]] = TensorDecl((E,), role="vector")
         for e in range(E):
             if spec.get("gated", True):
                 m[prefix + n["gate"].format(e=e)] = TensorDecl((ff, hid))
             m[prefix + n["up"].format(e=e)] = TensorDecl((ff, hid))
             m[prefix + n["down"].format(e=e)] = TensorDecl((hid, ff))
         if spec.get("shared_size"):
+            if spec.get("gated", True):
+                m[prefix + n["shared_gate"]] = TensorDecl((spec["shared_size"], hid))
             m[prefix + n["shared_up"]] = TensorDecl((spec["shared_size"], hid))
             m[prefix + n["shared_down"]] = TensorDecl((hid, spec["shared_size"]))
         return m
@@ -85,6 +93,13 @@ class MoEFeedForward(FeedForward):
         self.router_bias = None
         if n.get("router_bias"):
             self.router_bias = tensors[prefix + n["router_bias"]].to(device=dev, dtype=torch.float32).contiguous()
+        self.scores, self.group_top = str(spec.get("scores") or "softmax"), int(spec.get("group_top", 1))
+        self.router_scale = float(spec.get("router_scale", 1.0))
+        if self.scores not in ops.ROUTER_SCORES:
+            raise ValueError(f"unknown router scores {self.scores!r} (known: {', '.join(ops.ROUTER_SCORES)})")
+        self.correction = None
+        if n.get("correction"):
+            self.correction = tensors[prefix + n["correction"]].to(device=dev, dtype=torch.float32).contiguous()
         self.gated = bool(spec.get("gated", True))
         self.act_kind = str(spec.get("activation", "relu2"))
         if not self.gated and self.act_kind not in ops.ACTIVATIONS:
@@ -104,7 +119,14 @@ class MoEFeedForward(FeedForward):
         self.fused_act = self.act_kind if not self.gated and self.act_kind in ops.EPILOGUE_ACTIVATIONS else None
         self.down = torch.stack([get("down", e) for e in range(self.E)]).contiguous()
         self.shared_size = int(spec.get("shared_size") or 0)
-        if self.shared_size:
+        self.shared = None
+        if self.shared_size and self.gated:
+            if self.activation != (0.0, 1.0, 0.0):
+                raise ValueError("a shared expert beside gated experts has their plain silu form")
+            names = {"gate": n["shared_gate"], "up": n["shared_up"], "down": n["shared_down"]}
+            self.shared = SwiGLUFeedForward(PartSpec("swiglu", {"hidden_size": self.hidden, "intermediate_size": self.shared_size, "names": names}),
+                                            prefix, tensors, runtime)
+        elif self.shared_size:
             self.shared_up = Linear(tensors[prefix + n["shared_up"]], runtime)
             self.shared_down = Linear(tensors[prefix + n["shared_down"]], runtime)
 
@@ -118,7 +140,8 @@ class MoEFeedForward(FeedForward):
         n, dev, dt = step.n_tokens, x.device, self.runtime.dtype
         logits = self.router.forward(x, out_dtype=torch.float32)
         choice, weight = ops.moe_route(logits, self.top, self.renormalise, self.groups, self.keep_groups, self.renorm_eps,
-                                       bias=self.router_bias)
+                                       bias=self.router_bias, scores=self.scores, correction=self.correction,
+                                            group_top=self.group_top, scale=self.router_scale)
         if self.tensor_cores and n * self.top >= self.TENSOR_CORE_ROWS_PER_EXPERT * self.E and x.stride(0) % 8 == 0:
             # enough rows per expert to fill tiles of 128: both products on the tensor cores, the activation in the first one's epilogue
             pair_pos, list_rows, tile_group = ops.moe_plan(choice, self.E, 128, step.token_slot)
@@ -154,7 +177,9 @@ class MoEFeedForward(FeedForward):
                 ops.grouped_gemm(act, self.down, res, a_rows=None, tile_group=tile_group, tile_rows=tile)
         out = torch.empty((2 if self.shared_size else 1, n, self.hidden), dtype=torch.float32, device=dev)
         ops.moe_combine(res, pair_pos, weight, out[0])
-        if self.shared_size:
+        if self.shared is not None:
+            self.shared.forward_into(x, out[1][:x.shape[0]])
+        elif self.shared_size:
             # the expert every token takes: its down product writes the second float32 piece
             up = self.shared_up.forward(x)
             ops.activation(up, up, self.act_kind)

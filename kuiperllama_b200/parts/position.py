@@ -1,4 +1,4 @@
-"""Rotary position encoding: the table of inverse frequencies."""
+"""Position encodings: the tables of inverse frequencies of a rotation, and a sinusoid added to the embeddings."""
 from __future__ import annotations
 
 import math
@@ -93,3 +93,21 @@ class RotaryPosition(PositionEncoding):
 
     def rotary(self):
         return self.inv_freq, self.rotary_dim
+
+
+@register_position("sinusoidal")
+class SinusoidalPosition(PositionEncoding):
+    """A fixed sinusoid added to the embeddings before the first layer (Vaswani et al., "Attention Is All You Need", 2017):
+    entry 2i is sin(p f_i), entry 2i + 1 is cos(p f_i), f_i = base^(-2i / hidden).  The embedding kernel adds it; every frequency
+    comes as a float32 number and the rest of its float64 value, so that angles of long sequences keep their precision.
+    Spec: ``hidden_size``, ``base``.  The mixer behind it is handed no rotation."""
+
+    def __init__(self, spec, prefix, tensors, runtime: Runtime):
+        super().__init__(spec, prefix, tensors, runtime)
+        hidden, base = int(spec["hidden_size"]), float(spec["base"])
+        f = torch.tensor([base ** (-2.0 * i / hidden) for i in range((hidden + 1) // 2)], dtype=torch.float64)
+        high = f.to(torch.float32)
+        self.frequencies = torch.stack([high, (f - high.double()).to(torch.float32)]).contiguous().to(runtime.device)
+
+    def embedding_frequencies(self):
+        return self.frequencies

@@ -1,4 +1,4 @@
-"""The dense SwiGLU feed-forward."""
+"""The dense gated feed-forward (SwiGLU, or with another activation of the gate)."""
 from __future__ import annotations
 
 from typing import Dict
@@ -18,7 +18,8 @@ class SwiGLUFeedForward(FeedForward):
     (ExiledOfCode/KuiperLLama kuiper/source/model/llama3.cpp:692-718, swiglu_kernel.cu:18-21;
     gate = w1, up = w3, down = w2, tools/export_llama3.py:583-585).  Gate and up are stacked
     into one matrix at load (and the activation is applied in that product's epilogue where the
-    tensor-core kernel runs).  Spec: ``hidden_size``, ``intermediate_size``, ``names``."""
+    tensor-core kernel runs).  ``activation`` "gelu_tanh" puts the tanh form of gelu in silu's place.  Spec: ``hidden_size``,
+    ``intermediate_size``, ``activation`` ("silu"), ``names``."""
 
     accepts_lazy_norm = True
     may_accumulate = True
@@ -32,6 +33,9 @@ class SwiGLUFeedForward(FeedForward):
     def __init__(self, spec, prefix, tensors, runtime: Runtime):
         super().__init__(spec, prefix, tensors, runtime)
         self.hidden, self.inter = int(spec["hidden_size"]), int(spec["intermediate_size"])
+        self.activation = str(spec.get("activation") or "silu")
+        if self.activation not in ops.GATED_ACTIVATIONS:
+            raise ValueError(f"unknown activation {self.activation!r} (known: {', '.join(sorted(ops.GATED_ACTIVATIONS))})")
         n = spec["names"]
         dev, dt = runtime.device, runtime.dtype
         gate, up = (tensors[prefix + n[k]].to(device=dev, dtype=dt) for k in ("gate", "up"))
@@ -44,14 +48,21 @@ class SwiGLUFeedForward(FeedForward):
 
     def forward(self, x, step: StepContext):
         if isinstance(x, NormedLazy):
-            if self.fused and ops.stream_fusable(x.shape[0], self.gate_up.weight):
+            if self.fused and self.activation == "silu" and ops.stream_fusable(x.shape[0], self.gate_up.weight):
                 # gate, up and the activation in one kernel that also finishes the norm before them
                 act = ops.gemm_skinny_stream(self.gate_up.weight, x.scaled, row_scale=(x.ss, x.eps), swiglu=True)
                 return self.down.forward(act, allow_partials=True, sink=getattr(step, "residual_sink", None))
             x = x.dense()
+        return self.down.forward(self._activated(x), allow_partials=True, sink=getattr(step, "residual_sink", None))
+
+    def forward_into(self, x: torch.Tensor, out: torch.Tensor) -> None:
+        """The same into ``out`` (a tensor of the caller's, float32 or the compute dtype)."""
+        self.down.forward(self._activated(x), out=out)
+
+    def _activated(self, x: torch.Tensor) -> torch.Tensor:
         act = torch.empty((x.shape[0], self.inter), dtype=self.runtime.dtype, device=x.device)
         if self.fused:
-            ops.matmul_swiglu(x, self.gate_up.weight, act)
+            ops.matmul_swiglu(x, self.gate_up.weight, act, activation=self.activation)
         else:
-            ops.swiglu(self.gate_up.forward(x), act)
-        return self.down.forward(act, allow_partials=True, sink=getattr(step, "residual_sink", None))
+            ops.swiglu(self.gate_up.forward(x), act, activation=self.activation)
+        return act

@@ -1,8 +1,10 @@
 """Grouped-query attention over a window of recent keys, with the options that softmax attention in the plain
-Llama form does not have: biased projections, a norm on q and k heads, interleaved rotary pairs, values of
-another size, a sink, sigmoid weights, and pooled blocks before the window."""
+Llama form does not have: biased projections, a norm on q and k heads or over the whole projection, interleaved
+rotary pairs, values of another size, a sink, sigmoid weights, pooled blocks before the window, chunks, a bias by
+distance, and values mixed with another layer's."""
 from __future__ import annotations
 
+import math
 from typing import Dict, Optional
 
 import torch
@@ -13,6 +15,22 @@ from ..csrc import ops
 from ..weights.loader import TensorDecl
 from .base import Mixer, PositionEncoding, Runtime, StepContext, register_mixer
 from .linear import Linear, StackedInput
+
+
+def distance_buckets(distances: int, rows: int, largest: float) -> torch.Tensor:
+    """int64 [distances]: the row of a bias table of ``rows`` rows that distance n reads.  The first rows // 2 distances have a
+    row each; from there on the rows stand for distances that grow by a constant factor, the last row for ``largest`` and
+    everything beyond: half + floor(ln(n / half) / ln(largest / half) * (rows - half)), at most rows - 1."""
+    half = rows // 2
+    out = []
+    for n in range(distances):
+        if n < half:
+            out.append(n)
+        elif largest <= half:
+            out.append(rows - 1)
+        else:
+            out.append(min(rows - 1, half + int(math.floor(math.log(n / half) / math.log(largest / half) * (rows - half)))) if half else rows - 1)
+    return torch.tensor(out, dtype=torch.int64)
 
 
 @register_mixer("window_attention")
@@ -27,18 +45,29 @@ class WindowAttentionMixer(Mixer):
     learned number per head joins the denominator as exp(sink)) or "sigmoid": sigmoid(score + b_h) with
     ``names['head_bias']``, not normalised; head h reads kv head h // (H / KV); out = Wo on the heads side by side.
 
+    ``row_norm``: q and k are instead RMS-normed over their WHOLE projection before it is split into heads (``q_norm`` and
+    ``k_norm`` then hold a weight per row of the projection; no biases, no rotation).  ``chunk`` = C: token i sees the keys
+    j <= i of its own chunk of C positions, floor(i / C) = floor(j / C), counted from the sequence's first position.
+    ``distance_bias`` {"rows", "largest"}: with ``names['distance_bias']`` [rows, heads] the score gets
+    table[bucket(i - j), h] after the scaling (``distance_buckets``).  ``value_mix``: "keep" leaves the layer's values as
+    projected for later layers of the step; "mix" caches (1 - lambda) v + lambda v_kept, lambda = ``names['value_mix']``, one number.
+
     One product makes q | k | v; ``ops.qk_prepare`` does bias, rotation, norm and the cache write in one kernel;
-    ``ops.pool_blocks`` writes the means of the blocks that the step completes.  Softmax without pooled blocks
+    ``ops.qk_row_prepare`` does norm over rows, value mixing and cache write; ``ops.pool_blocks`` writes the means of the blocks
+    that the step completes.  Chunks, a distance bias and values of another size run on the tensor cores for bfloat16 key and
+    value sizes of 32, 64 and 128 (``ops.attention_chunked_mma``).  Softmax without pooled blocks
     runs on the attention kernels of ``AttentionMixer`` where they take the sizes; a sink, sigmoid weights and pooled blocks
     are options of the windowed tensor-core kernel (bfloat16, equal key and value sizes of 64 or 128, groups of up to 16
     heads); everything else runs on the plain kernels.
 
     Spec: ``hidden_size``, ``num_heads``, ``num_kv_heads``, ``head_dim``, ``value_dim``, ``scale``, ``window``, ``values``
-    ("own" | "keys"), ``weights`` ("softmax" | "sigmoid"), ``pool`` (None), ``head_norm`` (None | {"eps"}), ``names``
-    (q, k, o and optionally v, q_bias, k_bias, v_bias, q_norm, k_norm, sink, head_bias).  KuiperLLama's attention is
+    ("own" | "keys"), ``weights`` ("softmax" | "sigmoid"), ``pool`` (None), ``head_norm`` (None | {"eps"}), ``row_norm``
+    (None | {"eps"}), ``chunk``, ``distance_bias``, ``value_mix`` (None | "keep" | "mix"), ``names`` (q, k, o and optionally v,
+    q_bias, k_bias, v_bias, q_norm, k_norm, sink, head_bias, distance_bias, value_mix).  KuiperLLama's attention is
     the unbiased causal softmax over every earlier key (kuiper/source/model/llama3.cpp:610-639, mha_kernel.cu:61,74-106)."""
 
     KERNEL = "mma"                # "simt": the plain kernels also for bfloat16 (for comparisons)
+    chunk = 0                     # positions per chunk; 0: no chunks
 
     @classmethod
     def manifest(cls, spec: PartSpec, prefix: str) -> Dict[str, TensorDecl]:
@@ -52,9 +81,14 @@ class WindowAttentionMixer(Mixer):
         for key, size in (("q_bias", H * hd), ("k_bias", KV * hd), ("v_bias", KV * vd), ("sink", H), ("head_bias", H)):
             if n.get(key):
                 m[prefix + n[key]] = TensorDecl((size,), role="vector")
-        for key in ("q_norm", "k_norm"):
+        for key, heads in (("q_norm", H), ("k_norm", KV)):
             if n.get(key):
-                m[prefix + n[key]] = TensorDecl((hd,), role="vector", init="one_plus_normal")
+                size = heads * hd if spec.get("row_norm") is not None else hd
+                m[prefix + n[key]] = TensorDecl((size,), role="vector", init="one_plus_normal")
+        if spec.get("distance_bias") is not None:
+            m[prefix + n["distance_bias"]] = TensorDecl((spec["distance_bias"]["rows"], H), role="vector")
+        if spec.get("value_mix") == "mix":
+            m[prefix + n["value_mix"]] = TensorDecl((), role="vector")
         return m
 
     def __init__(self, spec, prefix, tensors, runtime: Runtime, position: Optional[PositionEncoding] = None):
@@ -75,7 +109,13 @@ class WindowAttentionMixer(Mixer):
         if self.weights not in ops.ATTENTION_WEIGHTS:
             raise ValueError(f"unknown attention weights {self.weights!r} (softmax, sigmoid)")
         self.scale = float(spec["scale"])
-        norm = spec.get("head_norm")
+        self.chunk = int(spec.get("chunk") or 0)
+        self.value_mix = spec.get("value_mix")
+        if self.value_mix not in (None, "keep", "mix"):
+            raise ValueError(f"unknown value mixing {self.value_mix!r} (keep, mix)")
+        row_norm = spec.get("row_norm")
+        self.by_rows = row_norm is not None or self.value_mix is not None      # prepared a whole projection at a time
+        norm = spec.get("head_norm") if not self.by_rows else row_norm
         self.head_norm, self.eps = norm is not None, float(norm["eps"]) if norm is not None else 0.0
         n = spec["names"]
         dev = runtime.device
@@ -83,6 +123,19 @@ class WindowAttentionMixer(Mixer):
         self.q_bias, self.k_bias, self.v_bias = f32("q_bias"), f32("k_bias"), f32("v_bias")
         self.q_norm, self.k_norm = f32("q_norm"), f32("k_norm")
         self.sink, self.head_bias = f32("sink"), f32("head_bias")
+        self.value_lambda = f32("value_mix").reshape(1) if self.value_mix == "mix" else None
+        self.distance_bias = None
+        if spec.get("distance_bias") is not None:
+            # a column per distance up to the largest one (or as far as a chunk or window reaches): what a key at that distance gets
+            rows, largest = int(spec["distance_bias"]["rows"]), float(spec["distance_bias"]["largest"])
+            reach = [int(math.ceil(max(largest, rows // 2))) + 1] + [int(c) for c in (self.chunk, self.window) if c]
+            table = f32("distance_bias")
+            self.distance_bias = table[distance_buckets(min(reach), rows, largest).to(dev)].T.contiguous()
+        if (self.chunk or self.distance_bias is not None) and (self.weights != "softmax" or self.pool or self.sink is not None):
+            raise ValueError("chunks and a distance bias go with a plain softmax: no sink, no sigmoid weights, no pooled blocks")
+        if self.by_rows and (self.values_are_keys or spec.get("head_norm") is not None or position is not None and position.rotary() is not None
+                             or any(t is not None for t in (self.q_bias, self.k_bias, self.v_bias))):
+            raise ValueError("a norm over the whole projection and mixed values come without biases, head norm, rotation and values that are keys")
         if self.sink is not None and self.weights != "softmax":
             raise ValueError("a sink joins a softmax's denominator; sigmoid weights have none")
         self.inputs = StackedInput(runtime)                 # q | k | v from one product
@@ -93,7 +146,7 @@ class WindowAttentionMixer(Mixer):
         self.o = Linear(tensors[prefix + n["o"]], runtime)
         rot = position.rotary() if position is not None else None
         self.inv_freq, self.rotary_dim = rot if rot is not None else (None, 0)
-        if position is not None and getattr(position, "magnitude", 1.0) != 1.0:
+        if rot is not None and getattr(position, "magnitude", 1.0) != 1.0:
             raise ValueError("this mixer's kernel rotates with unit magnitude")
         self.interleaved = getattr(position, "pairing", "half") == "interleaved"
 
@@ -101,11 +154,13 @@ class WindowAttentionMixer(Mixer):
         value_dim = None if self.vd == self.hd else self.vd
         if self.pool:
             return KVRequest(kv_heads=self.KV, head_dim=self.hd, kind="pooled", window=self.window, value_dim=value_dim, pool=self.pool)
-        return KVRequest(kv_heads=self.KV, head_dim=self.hd, kind="full", window=self.window, value_dim=value_dim)
+        return KVRequest(kv_heads=self.KV, head_dim=self.hd, kind="full", window=self.window, value_dim=value_dim, chunk=self.chunk or None)
 
     def forward(self, x, step: StepContext, cache: CacheView) -> torch.Tensor:
         if hasattr(x, "dense"):
             x = x.dense()
+        if self.by_rows or self.chunk or self.distance_bias is not None:
+            return self._forward_chunked(x, step, cache)
         n, dt = step.n_tokens, self.runtime.dtype
         proj = self.inputs.forward(x)
         q_col = self.inputs.column("q")
@@ -141,4 +196,53 @@ class WindowAttentionMixer(Mixer):
             ops.attention_pooled(q, attn, cache.k, cache.v, cache.block_table, step.positions, step.token_slot, n, self.H, self.KV,
                                  self.hd, self.vd, self.scale, window, weights=self.weights, sink=self.sink, head_bias=self.head_bias,
                                  pooled=cache.pooled if self.pool else None)
+        return self.o.forward(attn, allow_partials=True)
+
+    def _prepare(self, x, step: StepContext, cache: CacheView) -> torch.Tensor:
+        """The queries [n, H * head_dim], ready for the scores; keys and values are in the cache."""
+        n, dt = step.n_tokens, self.runtime.dtype
+        write = cache.writable
+        k_cache, v_cache = (cache.k, cache.v) if write else (None, None)
+        if not self.by_rows:
+            proj = self.inputs.forward(x)
+            q_col = self.inputs.column("q")
+            ops.qk_prepare(proj, q_col, self.inputs.column("k"), None if self.values_are_keys else self.inputs.column("v"),
+                           step.positions, step.token_slot, cache.block_table, k_cache, v_cache, n, self.H, self.KV, self.hd, self.vd,
+                           q_bias=self.q_bias, k_bias=self.k_bias, v_bias=self.v_bias, inv_freq=self.inv_freq, rotary_dim=self.rotary_dim,
+                           interleaved=self.interleaved, head_norm=self.head_norm, eps=self.eps, q_norm_weight=self.q_norm,
+                           k_norm_weight=self.k_norm)
+            return proj[:, q_col:q_col + self.H * self.hd]
+        proj = self.inputs.forward(x, allow_partials=True)          # few tokens: the product's pieces, which the kernel adds
+        make = torch.zeros if n > sum(step.host_new) else torch.empty
+        q = make((n, self.H * self.hd), dtype=dt, device=x.device)
+        keep = first = None
+        if self.value_mix == "keep":
+            keep = step.shared["values"] = make((n, self.KV * self.vd), dtype=dt, device=x.device)
+        elif self.value_mix == "mix":
+            first = step.shared["values"]
+        ops.qk_row_prepare(proj, self.inputs.column("q"), self.inputs.column("k"), self.inputs.column("v"), q, step, cache.block_table,
+                           k_cache, v_cache, self.H, self.KV, self.hd, self.vd, norm=self.head_norm, eps=self.eps, q_norm_weight=self.q_norm,
+                           k_norm_weight=self.k_norm, v_first=first, v_lambda=self.value_lambda, v_keep=keep)
+        return q
+
+    def _forward_chunked(self, x, step: StepContext, cache: CacheView) -> torch.Tensor:
+        n, dt = step.n_tokens, self.runtime.dtype
+        q = self._prepare(x, step, cache)
+        # rows that belong to no sequence (a small step's padding) are not written by the kernels: keep them defined
+        make = torch.zeros if n > sum(step.host_new) else torch.empty
+        attn = make((n, self.H * self.vd), dtype=dt, device=q.device)
+        window = int(self.window or 0)
+        if (dt == torch.bfloat16 and self.KERNEL == "mma" and self.hd in ops.CHUNKED_MMA_DIMS and self.vd in ops.CHUNKED_MMA_DIMS
+                and self.H // self.KV <= 16 and q.stride(0) % 2 == 0 and q.data_ptr() % 4 == 0):
+            splits = 1
+            if step.is_decode:
+                # never more pieces than the pages that a chunk or window spans
+                reach = [-(-int(r) // ops.PAGE) + 1 for r in (self.chunk, window) if r]
+                splits = min([ops.decode_attention_splits(step.n_seqs, self.KV, self.hd, getattr(step, "context_class", 0))] + reach)
+            ops.attention_chunked_mma(q, q.stride(0), attn, cache.k, cache.v, cache.block_table, step, self.H, self.KV, self.hd, self.vd,
+                                      self.scale, window=window, chunk=self.chunk, distance_bias=self.distance_bias, splits=splits,
+                                      few_rows=step.is_decode)
+        else:
+            ops.attention_simt(q, q.stride(0), attn, cache.k, cache.v, cache.block_table, step.positions, step.token_slot, n, self.H, self.KV,
+                               self.hd, self.scale, window, value_dim=self.vd, chunk=self.chunk, distance_bias=self.distance_bias)
         return self.o.forward(attn, allow_partials=True)
