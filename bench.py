@@ -4,8 +4,8 @@ B200, and the two other workloads of the same family (Llama-2-7B shape with ragg
 Llama-3.2-1B shape with temperature sampling).
 
     python bench.py [--gpus 1] [--steps K] [--warmup W] [--layers L] [--batch B] [--impl reference] [--no-points]
-    python bench.py --compare terolix|munadra|bededra|dofevik [--sizes 1b,8b-8-layers]   (another design beside Llama, Dofevik beside
-                                                                                         Munadra, the closest model; see compare_designs)
+    python bench.py --compare terolix|munadra|bededra|dofevik|vepolix [--sizes 1b,8b-8-layers]   (another design beside Llama, or beside the
+                                                 closest model: Dofevik beside Munadra, Vepolix beside Bededra; see compare_designs)
 
 A "step" is one decode step of a batch (default 8 sequences that each hold a 512-token
 prompt, context limit 4096).  One JSON line is printed:
@@ -432,6 +432,22 @@ def dofevik_config(width, layers, heads, kv_heads, head_dim, vocab):
             "layers": [dict(order[i % 4], mlp=moe) for i in range(layers)]}
 
 
+def vepolix_config(width, layers, heads, kv_heads, head_dim, vocab):
+    """A Vepolix model of ``layers`` layers in groups of four: a matrix memory (heads of 256 x 512, as many as make the width)
+    with a dense feed-forward of the Llama shape's intermediate size, attention in chunks of 1,024 (the Llama shape's heads, a
+    distance bias up to 128, mixed values), a matrix memory, and attention again; the last three with 16 experts in 4 groups
+    of which 2 are kept, 4 experts per token of a quarter of the Llama shape's intermediate size, and a shared expert of that size."""
+    inter = COMPARE_INTER[width]
+    mem = {"type": "mlstm", "mixer": {"heads": width // 512, "dim": 256, "vdim": 512, "gate_cap": 15.0}}
+    att = {"type": "attention", "mixer": {"heads": heads, "kv_heads": kv_heads, "dim": head_dim, "vdim": head_dim, "scale": head_dim ** -0.5,
+                                          "bias_max": 128, "mask": {"size": 1024}, "v_mix": True}}
+    moe = {"kind": "moe", "router": {"experts": 16, "top": 4, "groups": {"count": 4, "keep": 2}, "scale": 2.0}, "expert": {"ff": inter // 4},
+           "shared": {"ff": inter // 4}}
+    order = [dict(mem, mlp={"kind": "dense", "ff": inter}), dict(att, mlp=moe), dict(mem, mlp=moe), dict(att, mlp=moe)]
+    return {"architecture": "Vepolix", "vocab": vocab, "width": width, "norm": {"eps": 1e-5}, "embedding": {"scale": 1.0},
+            "layers": [order[i % 4] for i in range(layers)]}
+
+
 COMPARE_INTER = {2048: 8192, 4096: 14336}
 
 
@@ -445,7 +461,7 @@ COMPARE_SIZES = {
 
 
 def compare_designs(args):
-    """``--compare terolix`` (or ``munadra``, ``bededra``): prefill (one prompt of 2,048 tokens) and decode (8 and 64 sequences after
+    """``--compare terolix`` (or ``munadra``, ``bededra``, ``dofevik``, ``vepolix``): prefill (one prompt of 2,048 tokens) and decode (8 and 64 sequences after
     512-token prompts, CUDA graphs) of Terolix beside the Llama decoder at equal size, random weights,
     bfloat16.  Rates in tokens a second; ``hbm_frac`` is the weights' bytes over the decode step's time
     over the copy peak, ``tc_frac`` the prefill's matrix-product flops over its time over the bf16 peak."""
@@ -465,7 +481,7 @@ def compare_designs(args):
                      tie_word_embeddings=True)
         if args.compare == "munadra":
             other = munadra_config(z["width"], z["layers"], z["heads"], z["head_dim"], vocab)
-        elif args.compare == "bededra":
+        elif args.compare in ("bededra", "vepolix"):
             other = bededra_config(z["width"], z["layers"], z["heads"], z["kv_heads"], z["head_dim"], vocab)
         else:
             other = terolix_config(z["width"], z["layers"], z["heads"], z["kv_heads"], z["head_dim"], z["ff"], vocab)
@@ -473,17 +489,20 @@ def compare_designs(args):
         if args.compare == "dofevik":                     # beside the closest existing model: latent attention and experts
             base, llama = "munadra", munadra_config(z["width"], z["layers"], z["heads"], z["head_dim"], vocab)
             other = dofevik_config(z["width"], z["layers"], z["heads"], z["kv_heads"], z["head_dim"], vocab)
+        if args.compare == "vepolix":                     # beside the closest existing model: matrix recurrences, parallel blocks, grouped experts
+            base, llama = "bededra", other
+            other = vepolix_config(z["width"], z["layers"], z["heads"], z["kv_heads"], z["head_dim"], vocab)
         out[name] = {}
         for design, cfg in ((base, llama), (args.compare, other)):
             model = kl.random_model(config_from_dict(cfg), seed=0, dtype="bfloat16", device="cuda:0")
             infer = kl.Inference(model, max_tokens=64 * CONTEXT, max_batch=64, max_seq_len=CONTEXT)
             wbytes = model.weight_bytes()
             matrix_params = wbytes / 2 - vocab * z["width"]
-            if design in ("munadra", "bededra", "dofevik"):       # a token uses 4 of a layer's 16 experts: count what it multiplies by
+            if design in ("munadra", "bededra", "dofevik", "vepolix"):       # a token uses 4 of a layer's 16 experts: count what it multiplies by
                 moe_layers = sum(1 for l in cfg["layers"] if l["mlp"] and l["mlp"]["kind"] == "moe")
                 per_expert = (2 if design == "dofevik" else 3) * z["width"] * (COMPARE_INTER[z["width"]] // 4)   # no gate: two matrices
                 matrix_params -= moe_layers * 12 * per_expert
-            if design == "dofevik":
+            if design in ("dofevik", "vepolix"):
                 matrix_params -= vocab * z["width"]           # a classifier of its own, which runs on the wanted rows only
             t = time_prefill(infer, warmup=3, repeats=5, seed=2, checks=checks)
             r = {"weight_gb": round(wbytes / 1e9, 3), "prefill_tokens_per_s": round(PREFILL_LEN / t, 1), "prefill_ms": round(t * 1e3, 3),
@@ -532,8 +551,8 @@ def main():
     ap.add_argument("--dtype", default="bfloat16", choices=["bfloat16", "float32"])
     ap.add_argument("--no-points", action="store_true",
                     help="only the headline: skip the prefill, the batch 1, 64 and 128 points and the two other workloads")
-    ap.add_argument("--compare", default=None, choices=["terolix", "munadra", "bededra", "dofevik"],
-                    help="instead of the default workload: this design beside Llama (Dofevik: beside Munadra) at equal size (prefill and decode rates)")
+    ap.add_argument("--compare", default=None, choices=["terolix", "munadra", "bededra", "dofevik", "vepolix"],
+                    help="instead of the default workload: this design beside Llama (Dofevik: beside Munadra, Vepolix: beside Bededra) at equal size (prefill and decode rates)")
     ap.add_argument("--sizes", default="", help="with --compare: which of the sizes to run, with commas (default: all)")
     args = ap.parse_args()
     if args.impl == "reference":

@@ -45,6 +45,7 @@ SOURCES: Dict[str, str] = {
     "short_conv": "short_conv.cu",
     "outer_recurrence": "outer_recurrence.cu",
     "mlstm": "mlstm.cu",
+    "mlstm_chunked": "mlstm_chunked.cu",
     "attention_mixed": "attention_mixed.cu",
     "attention_mixed_tiled": "attention_mixed_tiled.cu",
     "qk_prepare": "qk_prepare.cu",

@@ -372,6 +372,128 @@ pair_rmsnorm_kernel(float* __restrict__ residual, const PairDelta d1, const Pair
     }
 }
 
+// The same with the row in registers and 8- or 16-byte accesses (rows of hidden % 4 == 0 elements up to 4 THREADS VPT whose
+// pointers and strides are aligned for it).
+template <typename T, int THREADS, int VPT>
+__global__ void __launch_bounds__(THREADS)
+pair_rmsnorm_vec_kernel(float* __restrict__ residual, const PairDelta d1, const PairDelta d2, const float* __restrict__ w1,
+                        const float* __restrict__ w2, float eps, T* __restrict__ out1, T* __restrict__ out2, const int* __restrict__ rows,
+                        int hidden) {
+    pdl_launch_dependents();
+    pdl_wait();
+    __shared__ float scratch[32];
+    const int r = blockIdx.x, n4 = hidden >> 2;
+    const size_t row = rows != nullptr ? (size_t)rows[r] : (size_t)r;
+    float* x = residual + row * hidden;
+    const bool has = d1.rows != nullptr || d1.pieces != nullptr || d2.rows != nullptr || d2.pieces != nullptr;
+    float4 v[VPT];
+    float ss = 0.f;
+    auto add_delta = [&](float4& a, const PairDelta& d, int i4) {
+        if (d.rows != nullptr) {
+            const float4 b = Vec4<T>::load((const T*)d.rows + row * d.ld + 4 * i4);
+            a.x += b.x; a.y += b.y; a.z += b.z; a.w += b.w;
+        }
+        for (int p0 = 0; p0 < d.n_pieces; p0 += 4) {           // four pieces on their way at a time, added in ascending order
+            float4 b[4];
+#pragma unroll
+            for (int p = 0; p < 4; ++p)
+                b[p] = p0 + p < d.n_pieces ? *reinterpret_cast<const float4*>(d.pieces + (size_t)(p0 + p) * d.piece_stride + row * hidden + 4 * i4)
+                                           : make_float4(0.f, 0.f, 0.f, 0.f);
+#pragma unroll
+            for (int p = 0; p < 4; ++p)
+                if (p0 + p < d.n_pieces) { a.x += b[p].x; a.y += b[p].y; a.z += b[p].z; a.w += b[p].w; }
+        }
+    };
+#pragma unroll
+    for (int j = 0; j < VPT; ++j) {
+        const int i4 = threadIdx.x + j * THREADS;
+        v[j] = make_float4(0.f, 0.f, 0.f, 0.f);
+        if (i4 < n4) {
+            v[j] = *reinterpret_cast<const float4*>(x + 4 * i4);
+            if (has) {
+                float4 a = make_float4(0.f, 0.f, 0.f, 0.f);
+                add_delta(a, d1, i4);
+                add_delta(a, d2, i4);
+                v[j].x += a.x; v[j].y += a.y; v[j].z += a.z; v[j].w += a.w;
+                if (rows == nullptr) *reinterpret_cast<float4*>(x + 4 * i4) = v[j];
+            }
+            ss += (v[j].x * v[j].x + v[j].y * v[j].y) + (v[j].z * v[j].z + v[j].w * v[j].w);
+        }
+    }
+    if (out1 == nullptr && out2 == nullptr) return;
+    ss = block_sum_once(ss, scratch);
+    const float inv = 1.0f / sqrtf(ss / (float)hidden + eps);
+#pragma unroll
+    for (int j = 0; j < VPT; ++j) {
+        const int i4 = threadIdx.x + j * THREADS;
+        if (i4 >= n4) continue;
+        const float4 y = make_float4(v[j].x * inv, v[j].y * inv, v[j].z * inv, v[j].w * inv);
+        if (out1 != nullptr) {
+            const float4 w = *reinterpret_cast<const float4*>(w1 + 4 * i4);
+            Vec4<T>::store(out1 + (size_t)r * hidden + 4 * i4, make_float4(y.x * w.x, y.y * w.y, y.z * w.z, y.w * w.w));
+        }
+        if (out2 != nullptr) {
+            const float4 w = *reinterpret_cast<const float4*>(w2 + 4 * i4);
+            Vec4<T>::store(out2 + (size_t)r * hidden + 4 * i4, make_float4(y.x * w.x, y.y * w.y, y.z * w.z, y.w * w.w));
+        }
+    }
+}
+
+// The per-head norm with the head in a warp's registers, four elements an access: heads of dim % 4 == 0 up to 128 VPL whose rows
+// are aligned for it.
+template <typename T, int VPL>
+__global__ void __launch_bounds__(128)
+head_rmsnorm_gate_vec_kernel(const float* __restrict__ x, const T* __restrict__ gate, long long gate_ld, const float* __restrict__ w,
+                             T* __restrict__ out, long long out_ld, float out_scale, int tokens, int heads, int dim, float eps, int gate_first,
+                             int wide_weight, const float* __restrict__ divisor, int sigmoid) {
+    pdl_launch_dependents();
+    pdl_wait();
+    const int lane = threadIdx.x & 31, n4 = dim >> 2;
+    const long long item = (long long)blockIdx.x * (blockDim.x >> 5) + (threadIdx.x >> 5);
+    if (item >= (long long)tokens * heads) return;
+    const int t = (int)(item / heads), h = (int)(item - (long long)t * heads);
+    const float* xr = x + ((size_t)t * heads + h) * dim;
+    const T* g = gate ? gate + (size_t)t * gate_ld + (size_t)h * dim : nullptr;
+    const float* wr = w != nullptr ? w + (wide_weight ? (size_t)h * dim : 0) : nullptr;
+    T* o = out + (size_t)t * out_ld + (size_t)h * dim;
+    const float pre = divisor != nullptr ? 1.0f / divisor[(size_t)t * heads + h] : 1.0f;
+    float4 v[VPL], f[VPL];
+    float ss = 0.f;
+#pragma unroll
+    for (int j = 0; j < VPL; ++j) {
+        const int i4 = lane + 32 * j;
+        v[j] = make_float4(0.f, 0.f, 0.f, 0.f);
+        f[j] = make_float4(1.f, 1.f, 1.f, 1.f);
+        if (i4 >= n4) continue;
+        v[j] = *reinterpret_cast<const float4*>(xr + 4 * i4);
+        if (g != nullptr) f[j] = Vec4<T>::load(g + 4 * i4);
+    }
+#pragma unroll
+    for (int j = 0; j < VPL; ++j) {
+        if (g != nullptr) {
+            f[j].x = gate_factor(f[j].x, sigmoid); f[j].y = gate_factor(f[j].y, sigmoid);
+            f[j].z = gate_factor(f[j].z, sigmoid); f[j].w = gate_factor(f[j].w, sigmoid);
+        }
+        v[j].x *= pre; v[j].y *= pre; v[j].z *= pre; v[j].w *= pre;
+        if (gate_first) { v[j].x *= f[j].x; v[j].y *= f[j].y; v[j].z *= f[j].z; v[j].w *= f[j].w; }
+        ss += (v[j].x * v[j].x + v[j].y * v[j].y) + (v[j].z * v[j].z + v[j].w * v[j].w);
+    }
+    ss = warp_sum(ss);
+    const float inv = 1.0f / sqrtf(ss / (float)dim + eps);
+#pragma unroll
+    for (int j = 0; j < VPL; ++j) {
+        const int i4 = lane + 32 * j;
+        if (i4 >= n4) continue;
+        float4 y = make_float4(v[j].x * inv, v[j].y * inv, v[j].z * inv, v[j].w * inv);
+        if (wr != nullptr) {
+            const float4 ww = *reinterpret_cast<const float4*>(wr + 4 * i4);
+            y.x *= ww.x; y.y *= ww.y; y.z *= ww.z; y.w *= ww.w;
+        }
+        if (!gate_first) { y.x *= f[j].x; y.y *= f[j].y; y.z *= f[j].z; y.w *= f[j].w; }
+        Vec4<T>::store(o + 4 * i4, make_float4(y.x * out_scale, y.y * out_scale, y.z * out_scale, y.w * out_scale));
+    }
+}
+
 }  // namespace kl
 
 using namespace kl;
@@ -440,6 +562,25 @@ KL_API int kl_head_rmsnorm_gate(const float* x, const void* gate, long long gate
     if (tokens <= 0 || heads <= 0) return KL_OK;
     if (dim <= 0) return KL_ERR_BAD_SIZE;
     const long long items = (long long)tokens * heads;
+    {   // heads that fit a warp's registers, on boundaries of four elements
+        const uintptr_t m = dtype == KL_BF16 ? 7 : 15;
+        if ((dtype == KL_F32 || dtype == KL_BF16) && dim % 4 == 0 && dim <= 1024 && gate_ld % 4 == 0 && out_ld % 4 == 0 &&
+            (((uintptr_t)gate | (uintptr_t)out) & m) == 0 && (((uintptr_t)x | (uintptr_t)w) & 15) == 0) {
+            const int blocks = (int)((items + 3) / 4);
+#define KL_HV(T, VPL)                                                                                                                    \
+    launch_kernel(head_rmsnorm_gate_vec_kernel<T, VPL>, blocks, 128, 0, stream, x, (const T*)gate, gate_ld, w, (T*)out, out_ld, out_scale, \
+                  tokens, heads, dim, eps, gate_first, wide_weight, divisor, sigmoid)
+#define KL_HV_BY(T)                                                                                                                      \
+    do {                                                                                                                                 \
+        if (dim <= 128) KL_HV(T, 1); else if (dim <= 256) KL_HV(T, 2); else if (dim <= 512) KL_HV(T, 4); else KL_HV(T, 8);               \
+    } while (0)
+            if (dtype == KL_F32) KL_HV_BY(float); else KL_HV_BY(bf16);
+#undef KL_HV_BY
+#undef KL_HV
+            KL_LAUNCH_CHECK();
+            return KL_OK;
+        }
+    }
     if (dim >= 512) {
         if (dtype == KL_F32)
             launch_kernel(head_rmsnorm_gate_block_kernel<float>, (int)items, dim >= 2048 ? 1024 : 256, 0, stream, x, (const float*)gate, gate_ld, w, (float*)out, out_ld, out_scale, heads, dim, eps, gate_first, wide_weight, divisor, sigmoid);
@@ -505,6 +646,30 @@ KL_API int kl_pair_rmsnorm(float* residual, const void* d1_rows, long long d1_ld
     if (hidden <= 0 || hidden > 48 * 1024 || (out1 != nullptr && w1 == nullptr) || (out2 != nullptr && w2 == nullptr)) return KL_ERR_BAD_SIZE;
     PairDelta a{d1_rows, d1_ld, d1_pieces, d1_pieces ? d1_n : 0, d1_stride};
     PairDelta b{d2_rows, d2_ld, d2_pieces, d2_pieces ? d2_n : 0, d2_stride};
+    if (dtype != KL_F32 && dtype != KL_BF16) return KL_ERR_BAD_DTYPE;
+    {   // the form with the row in registers, where everything is aligned for 8-byte (bfloat16) or 16-byte (float) accesses
+        const uintptr_t m = dtype == KL_BF16 ? 7 : 15;
+        const int n4 = hidden / 4;
+        auto ok_t = [&](const void* p, long long ld) { return p == nullptr || ((((uintptr_t)p) & m) == 0 && ld % 4 == 0); };
+        auto ok_f = [&](const void* p) { return (((uintptr_t)p) & 15) == 0; };
+        if (hidden % 4 == 0 && n4 <= 2048 && ok_t(d1_rows, d1_ld) && ok_t(d2_rows, d2_ld) && ok_t(out1, hidden) && ok_t(out2, hidden) &&
+            ok_f(residual) && ok_f(d1_pieces) && ok_f(d2_pieces) && ok_f(w1) && ok_f(w2)) {
+#define KL_PV(T, THREADS, VPT)                                                                                                            \
+    launch_kernel(pair_rmsnorm_vec_kernel<T, THREADS, VPT>, n_rows, THREADS, 0, stream, residual, a, b, w1, w2, eps, (T*)out1, (T*)out2, rows, hidden)
+#define KL_PV_BY(T)                                                                                                                       \
+    do {                                                                                                                                  \
+        /* few rows of a wide model (decode): a row over 512 or 1,024 threads, so that one round of loads fetches it */                    \
+        if (n_rows <= 256 && n4 > 256) { if (n4 <= 512) KL_PV(T, 512, 1); else if (n4 <= 1024) KL_PV(T, 1024, 1); else KL_PV(T, 1024, 2); } \
+        else if (n4 <= 64) KL_PV(T, 64, 1); else if (n4 <= 128) KL_PV(T, 128, 1); else if (n4 <= 256) KL_PV(T, 256, 1);                   \
+        else if (n4 <= 512) KL_PV(T, 256, 2); else if (n4 <= 1024) KL_PV(T, 512, 2); else KL_PV(T, 512, 4);                                \
+    } while (0)
+            if (dtype == KL_BF16) KL_PV_BY(bf16); else KL_PV_BY(float);
+#undef KL_PV_BY
+#undef KL_PV
+            KL_LAUNCH_CHECK();
+            return KL_OK;
+        }
+    }
     const size_t smem = (size_t)hidden * sizeof(float);
     // few rows: a row's loads (the stream, the rows or pieces of two results) are a chain per thread, so many threads
     const int pair_threads = n_rows <= 64 && hidden >= 2048 ? 1024 : 256;

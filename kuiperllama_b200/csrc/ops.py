@@ -1031,11 +1031,12 @@ def outer_recurrence(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, a: torch
         ctypes.c_float(den_eps), dtype_code(q.dtype), _stream()), "outer_recurrence")
 
 
-def mlstm_gates(x: torch.Tensor, weight: torch.Tensor, bias: torch.Tensor, cap: float, state: torch.Tensor, step):
+def mlstm_gates(x: torch.Tensor, weight: torch.Tensor, bias: torch.Tensor, cap: float, state: torch.Tensor, step, logs: bool = False):
     """The factors of a matrix memory with exponential gates (see mlstm.cu), float32 [rows, heads] each: (a, c, floor), from the
     log gates i = cap tanh(z_i / cap) and f = logsigmoid(cap tanh(z_f / cap)) with z = ``weight`` x + ``bias`` in 32 bits, and
     the running maximum in ``state`` (float32 [slots, >= heads]), which moves on.  ``weight`` [2 * heads, width] in the compute
-    dtype: the input gates' rows, then the forget gates'; ``bias`` float32 [2 * heads]."""
+    dtype: the input gates' rows, then the forget gates'; ``bias`` float32 [2 * heads].  With ``logs`` the result is instead float32
+    [4, rows, heads]: f, i, and the maximum before and after every token (what ``mlstm_chunked`` takes)."""
     _cuda(x, weight, bias, state)
     n, dev = step.n_tokens, x.device
     H, width = weight.shape[0] // 2, weight.shape[1]
@@ -1043,15 +1044,51 @@ def mlstm_gates(x: torch.Tensor, weight: torch.Tensor, bias: torch.Tensor, cap: 
     _need(weight.dtype == x.dtype and weight.is_contiguous() and weight.shape[0] == 2 * H, "mlstm_gates: weight [2 heads, width]")
     _need(bias.dtype == torch.float32 and bias.is_contiguous() and bias.numel() == 2 * H and cap > 0, "mlstm_gates: bias and cap")
     _need(state.dtype == torch.float32 and state.dim() == 2 and state.stride(1) == 1 and state.shape[1] >= H, "mlstm_gates: state")
-    single = bool(step.is_decode) and n == step.n_seqs
+    single = bool(step.is_decode) and n == step.n_seqs and not logs
     # rows that belong to no sequence (a small step's padding) are not written by the scan: keep them defined
-    a, c, floor = (torch.empty if single else torch.ones)((3, n, H), dtype=torch.float32, device=dev).unbind(0)
+    out = (torch.ones if step.padded else torch.empty)((4 if logs else 3, n, H), dtype=torch.float32, device=dev)
+    a, c, floor = (None, None, None) if logs else out.unbind(0)
     z = None if single else torch.empty((n, 2 * H), dtype=torch.float32, device=dev)
     _check(lib("mlstm").kl_mlstm_gates(
         _ptr(x), ctypes.c_longlong(x.stride(0)), _ptr(weight), width, _ptr(bias), ctypes.c_float(cap), _ptr(state),
-        ctypes.c_longlong(state.stride(0)), _ptr(z), _ptr(a), _ptr(c), _ptr(floor), _ptr(step.cu_tokens), _ptr(step.seq_slots), n,
+        ctypes.c_longlong(state.stride(0)), _ptr(z), _ptr(a), _ptr(c), _ptr(floor), _ptr(out if logs else None), _ptr(step.cu_tokens), _ptr(step.seq_slots), n,
         step.n_seqs, int(step.max_new), H, int(single), dtype_code(x.dtype), _stream()), "mlstm_gates", 1 if single else 2)
-    return a, c, floor
+    return out if logs else (a, c, floor)
+
+
+MLSTM_CHUNK = 64               # tokens per chunk; equals MC in mlstm_chunked.cu
+MLSTM_CHUNKED_FROM = 32        # tokens of the longest sequence from which a bfloat16 step takes the chunked form
+
+
+def mlstm_chunked_fits(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, dim: int, vdim: int) -> bool:
+    """Whether the chunked form takes these operands: bfloat16 rows on 16-byte boundaries, sizes that are multiples of 8, keys of
+    at most 256."""
+    return (q.dtype == k.dtype == v.dtype == torch.bfloat16 and dim % 8 == 0 and vdim % 8 == 0 and dim <= 256
+            and all(t.stride(0) % 8 == 0 and t.data_ptr() % 16 == 0 for t in (q, k, v)))
+
+
+def mlstm_chunked(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, logs: torch.Tensor, state: torch.Tensor, z_off: int, y: torch.Tensor,
+                  den: torch.Tensor, step, heads: int, dim: int, vdim: int, q_scale: float, den_eps: float) -> None:
+    """The matrix memory of a ragged step in chunks on the tensor cores (see mlstm_chunked.cu): y_t = S_t^T (q_scale q_t) float32
+    [rows, heads * vdim] and den_t = max(|z_t . q_scale q_t|, exp(-m_t)) + den_eps float32 [rows, heads], from and into ``state``
+    float32 [slots, ...]: S as [heads, dim, vdim], and z as [heads, dim] ``z_off`` elements behind it.  ``logs`` from
+    ``mlstm_gates(..., logs=True)``."""
+    _cuda(q, k, v, logs, state, y, den)
+    n = step.n_tokens
+    _columns(q, n, heads * dim, "mlstm_chunked: q"); _columns(k, n, heads * dim, "mlstm_chunked: k"); _columns(v, n, heads * vdim, "mlstm_chunked: v")
+    _need(mlstm_chunked_fits(q, k, v, dim, vdim), "mlstm_chunked: bfloat16 rows on 16-byte boundaries, sizes in multiples of 8, keys up to 256")
+    _need(logs.dtype == torch.float32 and logs.is_contiguous() and tuple(logs.shape) == (4, n, heads), "mlstm_chunked: logs")
+    _need(state.dtype == torch.float32 and state.dim() == 2 and state.stride(1) == 1 and state.shape[1] >= z_off + heads * dim
+          and z_off >= heads * dim * vdim, "mlstm_chunked: state")
+    for t, w in ((y, heads * vdim), (den, heads)):
+        _need(t.dtype == torch.float32 and t.is_contiguous() and t.shape[0] >= n and t.shape[1] == w, "mlstm_chunked: outputs")
+    chunks = -(-int(step.max_new) // MLSTM_CHUNK)
+    scratch = torch.empty(n * heads * (MLSTM_CHUNK + 2) + step.n_seqs * chunks * heads, dtype=torch.float32, device=q.device)
+    _check(lib("mlstm_chunked").kl_mlstm_chunked(
+        _ptr(q), ctypes.c_longlong(q.stride(0)), _ptr(k), ctypes.c_longlong(k.stride(0)), _ptr(v), ctypes.c_longlong(v.stride(0)), _ptr(logs),
+        _ptr(scratch), _ptr(state), ctypes.c_longlong(state.stride(0)), ctypes.c_longlong(z_off), _ptr(y), _ptr(den), _ptr(step.cu_tokens),
+        _ptr(step.seq_slots), n, step.n_seqs, int(step.max_new), heads, dim, vdim, ctypes.c_float(q_scale), ctypes.c_float(den_eps), _stream()),
+        "mlstm_chunked", 2)
 
 
 # --------------------------------------------------------------------------- attention with mixed heads

@@ -333,6 +333,78 @@ qk_row_prepare_kernel(const RowPrepare A) {
     }
 }
 
+// The same with one CTA per token: the token's q | k | v are cut into pieces of eight elements (bfloat16, 16-byte accesses), VPT
+// pieces a thread in registers, and one meeting of the warps adds both sums of squares.
+template <int VPT>
+__global__ void __launch_bounds__(512)
+qk_row_prepare_vec_kernel(const RowPrepare A) {
+    pdl_launch_dependents();
+    pdl_wait();
+    __shared__ float part[2][16];
+    const int t = blockIdx.x;
+    const int slot = A.token_slot[t];
+    if (slot < 0) return;                               // a padding row
+    const int pos = A.positions[t];
+    const int nq = A.H * A.hd / 8, nk = A.KV * A.hd / 8, nv = A.KV * A.vd / 8;
+    const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, nwarps = (blockDim.x + 31) >> 5;
+    float x[VPT][8];
+    float sq = 0.f, sk = 0.f;
+#pragma unroll
+    for (int j = 0; j < VPT; ++j) {
+        const int i = threadIdx.x + j * blockDim.x;
+        if (i >= nq + nk + nv) continue;
+        const int col = i < nq ? A.q_col + i * 8 : (i < nq + nk ? A.k_col + (i - nq) * 8 : A.v_col + (i - nq - nk) * 8);
+        rp_load<bf16, 8>(A, (size_t)t * A.ld + col, x[j]);
+        float ss = 0.f;
+#pragma unroll
+        for (int e = 0; e < 8; ++e) ss += x[j][e] * x[j][e];
+        if (i < nq) sq += ss;
+        else if (i < nq + nk) sk += ss;
+    }
+    float inv_q = 1.f, inv_k = 1.f;
+    if (A.norm) {
+        sq = warp_sum(sq);
+        sk = warp_sum(sk);
+        if (lane == 0) { part[0][warp] = sq; part[1][warp] = sk; }
+        __syncthreads();
+        sq = warp_sum(lane < nwarps ? part[0][lane] : 0.f);
+        sk = warp_sum(lane < nwarps ? part[1][lane] : 0.f);
+        inv_q = 1.0f / sqrtf(sq / (float)(nq * 8) + A.eps);
+        inv_k = 1.0f / sqrtf(sk / (float)(nk * 8) + A.eps);
+    }
+    const bool write = A.k_cache != nullptr;
+#pragma unroll
+    for (int j = 0; j < VPT; ++j) {
+        const int i = threadIdx.x + j * blockDim.x;
+        if (i >= nq + nk + nv) continue;
+        const bool is_q = i < nq, is_k = !is_q && i < nq + nk;
+        const int at = (is_q ? i : (is_k ? i - nq : i - nq - nk)) * 8;
+        if (is_q || is_k) {
+            const float* w = is_q ? A.q_w : A.k_w;
+            const float inv = is_q ? inv_q : inv_k;
+            if (w != nullptr) {
+                const float4 w0 = *reinterpret_cast<const float4*>(w + at), w1 = *reinterpret_cast<const float4*>(w + at + 4);
+                x[j][0] *= w0.x; x[j][1] *= w0.y; x[j][2] *= w0.z; x[j][3] *= w0.w; x[j][4] *= w1.x; x[j][5] *= w1.y; x[j][6] *= w1.z; x[j][7] *= w1.w;
+            }
+#pragma unroll
+            for (int e = 0; e < 8; ++e) x[j][e] *= inv;
+            if (is_q) rp_store<bf16, 8>((bf16*)A.q_out + (size_t)t * A.q_ld + at, x[j]);
+            else if (write) rp_store<bf16, 8>((bf16*)A.k_cache + cache_row_offset(A.block_table, A.blocks_per_seq, slot, pos, at / A.hd, A.KV, A.hd) + at % A.hd, x[j]);
+        } else {
+            if (A.v_keep != nullptr) rp_store<bf16, 8>((bf16*)A.v_keep + (size_t)t * nv * 8 + at, x[j]);
+            if (!write) continue;
+            if (A.v_first != nullptr) {
+                const float lam = A.lambda[0];
+                const uint4 raw = *reinterpret_cast<const uint4*>((const bf16*)A.v_first + (size_t)t * A.v_first_ld + at);
+                const bf16* f = reinterpret_cast<const bf16*>(&raw);
+#pragma unroll
+                for (int e = 0; e < 8; ++e) x[j][e] = (1.0f - lam) * x[j][e] + lam * to_f32(f[e]);
+            }
+            rp_store<bf16, 8>((bf16*)A.v_cache + cache_row_offset(A.block_table, A.blocks_per_seq, slot, pos, at / A.vd, A.KV, A.vd) + at % A.vd, x[j]);
+        }
+    }
+}
+
 }  // namespace kl
 
 using namespace kl;
@@ -357,6 +429,16 @@ KL_API int kl_qk_row_prepare(const void* rows, const float* pieces, int n_pieces
                            (uintptr_t)v_keep;
     const bool wide = dtype == KL_BF16 && hd % 8 == 0 && vd % 8 == 0 && ld % 8 == 0 && q_ld % 8 == 0 && v_first_ld % 8 == 0 && q_col % 8 == 0 &&
                       k_col % 8 == 0 && v_col % 8 == 0 && piece_stride % 8 == 0 && (ptrs & 15) == 0;
+    const int pieces8 = wide ? (H * hd + KV * hd + KV * vd) / 8 : 0;
+    if (wide && pieces8 <= 4 * 512 && (((uintptr_t)q_w | (uintptr_t)k_w) & 15) == 0) {
+        const int vpt = pieces8 <= 512 ? 1 : (pieces8 <= 1024 ? 2 : 4);
+        const int threads = ((pieces8 + vpt - 1) / vpt + 31) / 32 * 32;
+        if (vpt == 1) launch_kernel(qk_row_prepare_vec_kernel<1>, n_tokens, threads, 0, stream, A);
+        else if (vpt == 2) launch_kernel(qk_row_prepare_vec_kernel<2>, n_tokens, threads, 0, stream, A);
+        else launch_kernel(qk_row_prepare_vec_kernel<4>, n_tokens, threads, 0, stream, A);
+        KL_LAUNCH_CHECK();
+        return KL_OK;
+    }
     const dim3 grid(n_tokens, 3);
 #define KL_RP(T, V)                                                                                                                \
     do {                                                                                                                           \

@@ -147,17 +147,17 @@ class DecoderModel:
     def _weights(self):
         yield self.embedding
         yield self.lm_head.weight
-        for b in self.blocks:
-            for part in vars(b).values():
-                if not isinstance(part, Part):
-                    continue
-                for v in vars(part).values():
-                    if isinstance(v, torch.Tensor):
-                        yield v
-                    elif isinstance(v, Linear):
-                        yield v.weight
-                    elif isinstance(v, StackedInput):
-                        if v.linear is not None:
-                            yield v.linear.weight
-                        for _, w in v._pieces:
-                            yield w
+        parts = [p for b in self.blocks for p in vars(b).values() if isinstance(p, Part)]
+        for part in parts:                       # grows by the parts inside parts
+            for v in vars(part).values():
+                if isinstance(v, Part) and v not in parts:
+                    parts.append(v)
+                elif isinstance(v, torch.Tensor):
+                    yield v
+                elif isinstance(v, Linear):
+                    yield v.weight
+                elif isinstance(v, StackedInput):
+                    if v.linear is not None:
+                        yield v.linear.weight
+                    for _, w in v._pieces:
+                        yield w

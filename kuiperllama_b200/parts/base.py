@@ -70,6 +70,11 @@ class StepContext:
     # into theirs, for instance).  It starts empty with every step.
     shared: Dict[str, torch.Tensor] = field(default_factory=dict)
 
+    @property
+    def padded(self) -> bool:
+        """Whether the step has rows that belong to no sequence (kernels write nothing there)."""
+        return self.n_tokens > sum(self.host_new)
+
 
 @dataclass
 class StreamSink:

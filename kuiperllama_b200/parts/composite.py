@@ -59,7 +59,7 @@ class BranchMixer(Mixer):
         inputs, o = self._alone()
         inputs.forward(x)
         # rows that belong to no sequence (a small step's padding) are not written by the kernels: keep them defined
-        make = torch.empty if step.n_tokens == step.n_seqs else torch.zeros
+        make = torch.zeros if step.padded else torch.empty
         act = make((step.n_tokens, self.core_width), dtype=self.runtime.dtype, device=x.device)
         self.core(inputs, "", step, cache, act, 1.0)
         return o.forward(act, allow_partials=True)

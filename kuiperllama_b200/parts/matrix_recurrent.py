@@ -163,9 +163,12 @@ class MLSTMMixer(BranchMixer):
 
     then each head's o over its root mean square (over vdim) times a weight per channel, times sigmoid(Wg n), and the
     output projection.  The gates' projections, the gates, the maximum, S, z, o and the norm are 32-bit; the slot's state is S as
-    [heads, dim, vdim], z as [heads, dim] and m as [heads], float32.  Spec: ``hidden_size``, ``heads``, ``dim``, ``vdim``, ``cap``,
+    [heads, dim, vdim], z as [heads, dim] and m as [heads], float32.  bfloat16 steps with a sequence of
+    ``ops.MLSTM_CHUNKED_FROM`` tokens or more run in chunks on the tensor cores, everything else token by token.  Spec: ``hidden_size``, ``heads``, ``dim``, ``vdim``, ``cap``,
     ``q_scale``, ``den_eps``, ``norm_eps`` and ``names`` (q, k, v, g, o, norm, i, i_bias, f, f_bias).  KuiperLLama has no
     recurrent mixer (its mixer is mha_kernel.cu:61,74-106)."""
+
+    KERNEL = "chunked"            # "walk": token by token also for prompts (for comparisons)
 
     @classmethod
     def manifest(cls, spec: PartSpec, prefix: str) -> Dict[str, TensorDecl]:
@@ -207,12 +210,17 @@ class MLSTMMixer(BranchMixer):
 
     def core(self, stacked: StackedInput, tag: str, step: StepContext, cache: CacheView, out: torch.Tensor, out_scale: float) -> None:
         n, dev = step.n_tokens, out.device
-        a, c, floor = ops.mlstm_gates(stacked.rows, self.gate_weight, self.gate_bias, self.cap, cache.state[:, self.m_off:], step)
-        make = torch.empty if n == step.n_seqs else torch.zeros
-        o = make((n, self.H * self.dv), dtype=torch.float32, device=dev)
-        den = (torch.empty if n == step.n_seqs else torch.ones)((n, self.H), dtype=torch.float32, device=dev)
-        ops.outer_recurrence(stacked.view(tag + "q"), stacked.view(tag + "k"), stacked.view(tag + "v"), a, cache.state, o, step,
-                             self.H, self.H, self.d, self.dv, c=c, q_scale=self.q_scale,
-                             normaliser=(cache.state[:, self.z_off:], floor, den, self.den_eps))
+        q, k, v = (stacked.view(tag + name) for name in ("q", "k", "v"))
+        # rows that belong to no sequence (a small step's padding) are not written by the kernels: keep them defined
+        o = (torch.zeros if step.padded else torch.empty)((n, self.H * self.dv), dtype=torch.float32, device=dev)
+        den = (torch.ones if step.padded else torch.empty)((n, self.H), dtype=torch.float32, device=dev)
+        maxima = cache.state[:, self.m_off:]
+        if self.KERNEL == "chunked" and step.max_new >= ops.MLSTM_CHUNKED_FROM and ops.mlstm_chunked_fits(q, k, v, self.d, self.dv):
+            logs = ops.mlstm_gates(stacked.rows, self.gate_weight, self.gate_bias, self.cap, maxima, step, logs=True)
+            ops.mlstm_chunked(q, k, v, logs, cache.state, self.z_off, o, den, step, self.H, self.d, self.dv, self.q_scale, self.den_eps)
+        else:
+            a, c, floor = ops.mlstm_gates(stacked.rows, self.gate_weight, self.gate_bias, self.cap, maxima, step)
+            ops.outer_recurrence(q, k, v, a, cache.state, o, step, self.H, self.H, self.d, self.dv, c=c, q_scale=self.q_scale,
+                                 normaliser=(cache.state[:, self.z_off:], floor, den, self.den_eps))
         ops.head_rmsnorm_gate(o, stacked.view(tag + "g"), self.norm_weight, out, self.H, self.dv, self.norm_eps, out_scale=out_scale,
                               divisor=den, gate_act="sigmoid")

@@ -173,7 +173,7 @@ class WindowAttentionMixer(Mixer):
         if self.pool and write:
             ops.pool_blocks(cache.k, cache.v, cache.block_table, cache.pooled, step, self.KV, self.hd, self.vd)
         # rows that belong to no sequence (a small step's padding) are not written by the kernels: keep them defined
-        make = torch.zeros if n > sum(step.host_new) else torch.empty
+        make = torch.zeros if step.padded else torch.empty
         attn = make((n, self.H * self.vd), dtype=dt, device=proj.device)
         q = proj[:, q_col:q_col + self.H * self.hd]
         window = int(self.window or 0)
@@ -213,7 +213,7 @@ class WindowAttentionMixer(Mixer):
                            k_norm_weight=self.k_norm)
             return proj[:, q_col:q_col + self.H * self.hd]
         proj = self.inputs.forward(x, allow_partials=True)          # few tokens: the product's pieces, which the kernel adds
-        make = torch.zeros if n > sum(step.host_new) else torch.empty
+        make = torch.zeros if step.padded else torch.empty
         q = make((n, self.H * self.hd), dtype=dt, device=x.device)
         keep = first = None
         if self.value_mix == "keep":
@@ -229,7 +229,7 @@ class WindowAttentionMixer(Mixer):
         n, dt = step.n_tokens, self.runtime.dtype
         q = self._prepare(x, step, cache)
         # rows that belong to no sequence (a small step's padding) are not written by the kernels: keep them defined
-        make = torch.zeros if n > sum(step.host_new) else torch.empty
+        make = torch.zeros if step.padded else torch.empty
         attn = make((n, self.H * self.vd), dtype=dt, device=q.device)
         window = int(self.window or 0)
         if (dt == torch.bfloat16 and self.KERNEL == "mma" and self.hd in ops.CHUNKED_MMA_DIMS and self.vd in ops.CHUNKED_MMA_DIMS
