@@ -163,6 +163,7 @@ class ParallelMixer(Mixer):
         o = torch.zeros((self.branches[0].o_weight.shape[0], width), dtype=dt, device=dev)
         for p, at in zip(self.branches, self.offsets):
             o[:, at:at + p.core_width] = p.o_weight.to(device=dev, dtype=dt)
+            p.o_weight = None                                  # its columns of the shared matrix are the only copy
         self.o = Linear(o, runtime)
 
     def kv_request(self) -> Optional[KVRequest]:

@@ -88,22 +88,28 @@ def attention(h: torch.Tensor, m: dict, w: Dict[str, torch.Tensor], eps: float, 
     return torch.einsum("hij,jhd->ihd", p, v).reshape(n, H * dv) @ w["o"].T, own
 
 
-def mlstm_recurrence(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, i: torch.Tensor, f: torch.Tensor) -> torch.Tensor:
-    """q, k [n, d] and v [n, dv] of one head, log gates i, f [n] -> [n, dv].  S, n and m start at zero:
-    m' = max(f + m, i);  S' = exp(f + m - m') S + exp(i - m') k v^T;  n' likewise with k alone;
-    o = S'^T q / (max(|n' . q|, exp(-m')) + 1e-6)."""
+def mlstm_sums(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, i: torch.Tensor, f: torch.Tensor) -> Tuple[torch.Tensor, torch.Tensor]:
+    """q, k [n, d] and v [n, dv] of one head, log gates i, f [n] -> (S'^T q [n, dv], max(|n' . q|, exp(-m')) + 1e-6 [n]).
+    S, n and m start at zero:  m' = max(f + m, i);  S' = exp(f + m - m') S + exp(i - m') k v^T;  n' likewise with k alone."""
     S = torch.zeros(k.shape[1], v.shape[1], dtype=F)
     z = torch.zeros(k.shape[1], dtype=F)
     m = torch.zeros((), dtype=F)
-    out = []
+    num, den = [], []
     for t in range(q.shape[0]):
         m_new = torch.maximum(f[t] + m, i[t])
         keep, take = torch.exp(f[t] + m - m_new), torch.exp(i[t] - m_new)
         S = keep * S + take * torch.outer(k[t], v[t])
         z = keep * z + take * k[t]
         m = m_new
-        out.append(S.T @ q[t] / (torch.maximum((z @ q[t]).abs(), torch.exp(-m)) + 1e-6))
-    return torch.stack(out)
+        num.append(S.T @ q[t])
+        den.append(torch.maximum((z @ q[t]).abs(), torch.exp(-m)) + 1e-6)
+    return torch.stack(num), torch.stack(den)
+
+
+def mlstm_recurrence(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, i: torch.Tensor, f: torch.Tensor) -> torch.Tensor:
+    """[n, dv]: one head's output, the sum over the denominator."""
+    num, den = mlstm_sums(q, k, v, i, f)
+    return num / den[:, None]
 
 
 def log_gates(h: torch.Tensor, w: Dict[str, torch.Tensor], cap: float) -> Tuple[torch.Tensor, torch.Tensor]:
