@@ -40,6 +40,7 @@ struct OuterArgs {
     float* y; long long ld_y;                        // [rows, heads * P]
     const int* cu_tokens; const int* seq_slots;
     int heads, groups, N, P, L, a_per_row;
+    int tile;                                        // tokens per shared-memory tile (the lane form; OR_TILE unless the rows are long)
     int vec_state;                                   // every row piece of four columns of S is 16-byte aligned
     int vec_in;                                      // k, q and a can be read four elements at a time
     float q_scale;
@@ -91,8 +92,8 @@ outer_recurrence_kernel(const OuterArgs A) {
     }
     const TI* qp = (const TI*)A.q; const TI* kp = (const TI*)A.k; const TI* vp = (const TI*)A.v;
     const float skip = A.skip != nullptr ? A.skip[h] : 0.f;
-    for (int t0 = 0; t0 < n_new; t0 += OR_TILE) {
-        const int nt = min(OR_TILE, n_new - t0);
+    for (int t0 = 0; t0 < n_new; t0 += A.tile) {
+        const int nt = min(A.tile, n_new - t0);
         __syncthreads();
         // the tile's k (times c), q (times q_scale), a and v, each in a loop of its own so that the loads of several
         // turns are in flight together
@@ -481,7 +482,10 @@ KL_API int kl_outer_recurrence(const void* q, long long ld_q, int q_col, const v
     while (threads > 128 && (threads / 2 >= P * L || (long long)((P * L + threads - 1) / threads) * heads * n_seqs < 2LL * sms)) threads >>= 1;
     const int cols = threads / L;
     dim3 grid((P + cols - 1) / cols, heads, n_seqs);
-    const size_t smem = (size_t)OR_TILE * (2 * N + (a_per_row ? N : 1) + cols) * sizeof(float);
+    const size_t per_token = (size_t)(2 * N + (a_per_row ? N : 1) + cols) * sizeof(float);
+    A.tile = OR_TILE;
+    while (A.tile > 1 && A.tile * per_token > 200 * 1024) A.tile >>= 1;
+    const size_t smem = A.tile * per_token;
     if (smem > 200 * 1024) return KL_ERR_BAD_SIZE;
 #define KL_OR_N(TI, NPT, NM)                                                                                        \
     do {                                                                                                            \

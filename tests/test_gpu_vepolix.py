@@ -264,7 +264,7 @@ def _memory_plain(q, k, v, x, W, b, cap, news, H, d, dv):
 @pytest.mark.parametrize("form, dtype", [("walk", "float32"), ("walk", "bfloat16"), ("chunked", "bfloat16")])
 @pytest.mark.parametrize("H, d, dv, f_bias, i_bias, cap", [(3, 8, 12, 2.0, 0.0, 9.0), (2, 24, 10, 3.0, 1.0, 4.0), (1, 256, 72, 2.0, 0.0, 12.0), (3, 128, 64, 6.0, 0.0, 12.0),
                                                             (4, 64, 96, 2.0, -4.0, 15.0), (2, 40, 8, -8.0, 0.0, 12.0), (2, 200, 24, 9.0, 6.0, 12.0),
-                                                            (3, 7, 5, 2.0, 0.0, 9.0), (1, 33, 9, 5.0, 0.0, 6.0), (2, 300, 16, 2.0, 0.0, 8.0), (2, 6, 512, 2.0, 0.0, 8.0)])
+                                                            (3, 7, 5, 2.0, 0.0, 9.0), (1, 33, 9, 5.0, 0.0, 6.0), (2, 300, 16, 2.0, 0.0, 8.0), (1, 1000, 6, 2.0, 0.0, 8.0), (2, 6, 512, 2.0, 0.0, 8.0)])
 def test_the_memory_over_ragged_portions(form, dtype, H, d, dv, f_bias, i_bias, cap):
     """Gates, running maximum, matrix, normaliser and denominator alone: sequences of several lengths in portions of many sizes
     (single tokens, portions shorter and longer than a chunk, ends at a chunk's border and one off), gates that forget nearly all
