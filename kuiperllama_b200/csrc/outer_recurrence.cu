@@ -17,6 +17,8 @@
 //       lanes' sums are added by shuffles.  Tokens are walked in order from the slot's state, so a result does not
 //       depend on how a prompt was cut.
 //   outer_recurrence_slab_kernel<TI, R, C>   the form that runs where the sizes allow: R x C of S per thread (see there).
+//   outer_recurrence_single_kernel<TI, CL>   a step of single tokens, bound by reading and writing S once: neighbouring lanes hold
+//       neighbouring columns of a row, eight rows a thread on their way at a time.
 //   decay_softplus_kernel     dt = softplus(raw + bias), a = exp(-exp(A_log) dt) per (token, head), 32-bit.
 //   decay_lowrank_kernel      a = sigmoid(z)^(1 / tau) = exp(-softplus(-z) / tau), z = W2 r + b with r a short row per
 //                             token (the first of two projections, made with the mixer's other projections), 32-bit.
@@ -352,6 +354,83 @@ outer_recurrence_slab_kernel(const OuterArgs A) {
     }
 }
 
+// One token per sequence.  A CTA takes 4 CL columns of S of one (sequence, head); CL lanes hold four columns each and
+// OS_THREADS / CL groups of lanes share the rows.
+constexpr int OS_THREADS = 256;
+template <typename TI, int CL>
+__global__ void __launch_bounds__(OS_THREADS)
+outer_recurrence_single_kernel(const OuterArgs A) {
+    pdl_launch_dependents();
+    pdl_wait();
+    constexpr int RG = OS_THREADS / CL, U = 8;
+    extern __shared__ __align__(16) float sm[];
+    __shared__ float scratch[33];
+    const int s = blockIdx.z, h = blockIdx.y, N = A.N, P = A.P;
+    if (A.cu_tokens[s + 1] <= A.cu_tokens[s]) return;
+    const size_t row = (size_t)A.cu_tokens[s];
+    const int g = h / (A.heads / A.groups);
+    float* kk = sm;                                            // [N] times c
+    float* qq = kk + N;                                        // [N] times q_scale
+    float* aa = qq + N;                                        // [N]
+    float* part = aa + N;                                      // [RG][4 CL]; N is a multiple of 4
+    const int cl = threadIdx.x % CL, rg = threadIdx.x / CL;
+    const int col = (blockIdx.x * CL + cl) * 4;
+    const bool live = col < P;                                 // P is a multiple of 4
+    float* S = A.state + (size_t)A.seq_slots[s] * A.ld_state + (size_t)h * N * P + col;
+    const float c = A.c != nullptr ? A.c[row * A.ld_c + h] : 1.f;
+    for (int n = threadIdx.x; n < N; n += OS_THREADS) {
+        kk[n] = to_f32(((const TI*)A.k)[row * A.ld_k + A.k_col + (size_t)g * N + n]) * c;
+        qq[n] = to_f32(((const TI*)A.q)[row * A.ld_q + A.q_col + (size_t)g * N + n]) * A.q_scale;
+        aa[n] = A.a_per_row ? A.a[row * A.ld_a + (size_t)h * N + n] : A.a[row * A.ld_a + h];
+    }
+    float v[4] = {0.f, 0.f, 0.f, 0.f}, acc[4] = {0.f, 0.f, 0.f, 0.f};
+    if (live) {
+#pragma unroll
+        for (int j = 0; j < 4; ++j) v[j] = to_f32(((const TI*)A.v)[row * A.ld_v + A.v_col + (size_t)h * P + col + j]);
+    }
+    __syncthreads();
+    for (int n0 = rg; n0 < N && live; n0 += RG * U) {
+        float4 x[U];
+#pragma unroll
+        for (int u = 0; u < U; ++u) {
+            const int n = n0 + u * RG;
+            x[u] = n < N ? *reinterpret_cast<const float4*>(S + (size_t)n * P) : make_float4(0.f, 0.f, 0.f, 0.f);
+        }
+#pragma unroll
+        for (int u = 0; u < U; ++u) {
+            const int n = n0 + u * RG;
+            if (n >= N) break;
+            const float kn = kk[n], qn = qq[n], an = aa[n];
+            x[u].x = fmaf(an, x[u].x, kn * v[0]); x[u].y = fmaf(an, x[u].y, kn * v[1]);
+            x[u].z = fmaf(an, x[u].z, kn * v[2]); x[u].w = fmaf(an, x[u].w, kn * v[3]);
+            acc[0] = fmaf(x[u].x, qn, acc[0]); acc[1] = fmaf(x[u].y, qn, acc[1]);
+            acc[2] = fmaf(x[u].z, qn, acc[2]); acc[3] = fmaf(x[u].w, qn, acc[3]);
+            *reinterpret_cast<float4*>(S + (size_t)n * P) = x[u];
+        }
+    }
+    *reinterpret_cast<float4*>(part + (size_t)rg * 4 * CL + 4 * cl) = make_float4(acc[0], acc[1], acc[2], acc[3]);
+    __syncthreads();
+    if (threadIdx.x < 4 * CL && blockIdx.x * 4 * CL + threadIdx.x < P) {
+        const int at = blockIdx.x * 4 * CL + threadIdx.x;
+        float y = 0.f;
+#pragma unroll
+        for (int r = 0; r < RG; ++r) y += part[r * 4 * CL + threadIdx.x];
+        if (A.skip != nullptr) y = fmaf(A.skip[h], to_f32(((const TI*)A.v)[row * A.ld_v + A.v_col + (size_t)h * P + at]), y);
+        A.y[row * A.ld_y + (size_t)h * P + at] = y;
+    }
+    if (A.norm_state != nullptr && blockIdx.x == 0) {          // the normaliser: the first columns' CTA
+        float* z = A.norm_state + (size_t)A.seq_slots[s] * A.ld_state + (size_t)h * N;
+        float dot = 0.f;
+        for (int n = threadIdx.x; n < N; n += OS_THREADS) {
+            const float x = fmaf(aa[n], z[n], kk[n]);
+            z[n] = x;
+            dot = fmaf(x, qq[n], dot);
+        }
+        dot = block_sum(dot, scratch);
+        if (threadIdx.x == 0) A.den[row * A.heads + h] = or_den(A, row, h, dot);
+    }
+}
+
 __global__ void decay_softplus_kernel(const void* __restrict__ raw, long long ld_raw, int col, int bf, const float* __restrict__ bias,
                                       const float* __restrict__ A_log, int rows, int heads, float* __restrict__ dt,
                                       float* __restrict__ a) {
@@ -414,6 +493,22 @@ KL_API int kl_outer_recurrence(const void* q, long long ld_q, int q_col, const v
     A.a_per_row = a_per_row ? 1 : 0; A.q_scale = q_scale;
     A.norm_state = norm_state; A.floor = floor; A.den = den; A.den_eps = den_eps;
     A.vec_state = ((uintptr_t)state % 16 == 0 && ld_state % 4 == 0 && P % 4 == 0) ? 1 : 0;
+    // single tokens: S read and written once
+    if (max_new == 1 && A.vec_state && N % 4 == 0 && N <= 1024) {
+        const bool narrow = (long long)((P + 127) / 128) * heads * n_seqs < 2LL * sms;
+        const int cols = narrow ? 64 : 128;
+        const dim3 grid((P + cols - 1) / cols, heads, n_seqs);
+        const size_t smem = (size_t)(3 * N + 4 * OS_THREADS) * sizeof(float);
+        if (in_dtype == KL_F32) {
+            if (narrow) launch_kernel(outer_recurrence_single_kernel<float, 16>, grid, OS_THREADS, smem, stream, A);
+            else launch_kernel(outer_recurrence_single_kernel<float, 32>, grid, OS_THREADS, smem, stream, A);
+        } else {
+            if (narrow) launch_kernel(outer_recurrence_single_kernel<bf16, 16>, grid, OS_THREADS, smem, stream, A);
+            else launch_kernel(outer_recurrence_single_kernel<bf16, 32>, grid, OS_THREADS, smem, stream, A);
+        }
+        KL_LAUNCH_CHECK();
+        return KL_OK;
+    }
     {   // slabs of R x C in registers: the largest slab that still gives every SM eight warps, else the smallest that fits
         const int slabs[3][2] = {{8, 4}, {4, 4}, {2, 2}};
         int pick = -1, pick_lr = 0;
