@@ -8,7 +8,8 @@ from .munadra import MunadraConfig
 from .bededra import BededraConfig
 from .dofevik import DofevikConfig
 from .vepolix import VepolixConfig
+from .voserax import VoseraxConfig
 
 __all__ = ["ConfigError", "config_class", "config_from_dict", "config_from_file", "config_from_folder",
            "known_architectures", "register_architecture", "LayerSpec", "ModelSpec", "PartSpec",
-           "ScheduleEntry", "default_schedule", "Llama3RopeScaling", "LlamaConfig", "TerolixConfig", "MunadraConfig", "BededraConfig", "DofevikConfig", "VepolixConfig"]
+           "ScheduleEntry", "default_schedule", "Llama3RopeScaling", "LlamaConfig", "TerolixConfig", "MunadraConfig", "BededraConfig", "DofevikConfig", "VepolixConfig", "VoseraxConfig"]

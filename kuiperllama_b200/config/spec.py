@@ -46,13 +46,17 @@ class LayerSpec:
     feed_forward_post_norm: Optional[PartSpec] = None
     mixer_gate: Optional[PartSpec] = None
     feed_forward_gate: Optional[PartSpec] = None
+    # What the arrangement "streams" has: how each sublayer reads and writes several residual streams.
+    mixer_streams: Optional[PartSpec] = None
+    feed_forward_streams: Optional[PartSpec] = None
 
     def parts(self):
         """(family, attribute, spec) of every part the layer has, in the order they are built."""
         out = [("norm", "mixer_norm", self.mixer_norm), ("mixer", "mixer", self.mixer),
                ("norm", "feed_forward_norm", self.feed_forward_norm), ("feed_forward", "feed_forward", self.feed_forward),
                ("norm", "mixer_post_norm", self.mixer_post_norm), ("norm", "feed_forward_post_norm", self.feed_forward_post_norm),
-               ("gate", "mixer_gate", self.mixer_gate), ("gate", "feed_forward_gate", self.feed_forward_gate)]
+               ("gate", "mixer_gate", self.mixer_gate), ("gate", "feed_forward_gate", self.feed_forward_gate),
+               ("streams", "mixer_streams", self.mixer_streams), ("streams", "feed_forward_streams", self.feed_forward_streams)]
         return [(f, a, s) for f, a, s in out if s is not None]
 
 
@@ -80,6 +84,7 @@ class ModelSpec:
     ignorable_suffixes: Tuple[str, ...] = ()
     # Options that some decoders have around the layers; None leaves the step out.
     embedding_multiplier: Optional[float] = None     # x = multiplier * E[token]
+    embedding_position: Optional[PartSpec] = None    # a position encoding that is added to the embeddings (None: what the first layer's adds)
     logit_scale: Optional[float] = None              # logits = scale * (W_cls x)
     logit_softcap: Optional[float] = None            # logits = cap * tanh(logits / cap), after the scale
 

@@ -66,7 +66,7 @@ struct GemmArgs {
     // With swiglu and act_custom: min(g, limit) * sigmoid(alpha * min(g, limit)) * (clamp(u, -limit, limit) + shift),
     // no clamp when limit <= 0 (act_custom 0: silu(g) * u).  With act_cubic c the sigmoid's argument is
     // alpha * g * (1 + c g^2): with alpha = 2 sqrt(2 / pi) and c = 0.044715 that is the tanh form of gelu, since
-    // (1 + tanh(y)) / 2 = sigmoid(2 y).
+    // (1 + tanh(y)) / 2 = sigmoid(2 y).  act_custom 2: max(g, 0) * u.
     int act_custom;
     float act_limit, act_alpha, act_shift, act_cubic;
     // The plain epilogue's activation on a complete result in bfloat16 (grouped products, no k cuts): 0 none, 1 the
@@ -98,6 +98,7 @@ __device__ __forceinline__ float plain_act(const GemmArgs& args, float y) {
 }
 __device__ __forceinline__ float gated_mul(const GemmArgs& args, float g, float u) {
     if (!args.act_custom) return silu_mul(g, u);
+    if (args.act_custom == 2) return fmaxf(g, 0.f) * u;
     if (args.act_limit > 0.f) { g = fminf(g, args.act_limit); u = fminf(fmaxf(u, -args.act_limit), args.act_limit); }
     return __fdividef(g, 1.0f + __expf(-args.act_alpha * g * fmaf(args.act_cubic * g, g, 1.0f))) * (u + args.act_shift);
 }
@@ -720,9 +721,13 @@ static int launch_pairs(const CUtensorMap& ma, const CUtensorMap& mb, const Gemm
     return KL_OK;
 }
 
-// The gated epilogue by name: 0 none, 1 silu(g) * u, 2 gelu(g) * u in its tanh form.
-static void set_gated(GemmArgs& args, int kind) {
+// The gated epilogue by number: 0 none, 1 silu(g) * u, 2 gelu(g) * u in its tanh form, 3 relu(g) * u, 4 the clamped form of
+// (limit, alpha, shift) (see GemmArgs).
+constexpr int GATED_KINDS = 4;
+static void set_gated(GemmArgs& args, int kind, float limit, float alpha, float shift) {
     args.swiglu = kind != 0;
+    if (kind == 3) args.act_custom = 2;
+    if (kind == 4) { args.act_custom = 1; args.act_limit = limit; args.act_alpha = alpha; args.act_shift = shift; args.act_cubic = 0.f; }
     if (kind == 2) { args.act_custom = 1; args.act_limit = 0.f; args.act_alpha = 1.5957691216057308f; args.act_shift = 0.f; args.act_cubic = 0.044715f; }
 }
 
@@ -736,11 +741,11 @@ using namespace kl;
 
 // out[M, N] = a[M, K] * w[N, K]^T, tokens as tile rows (any M).  out is bf16 (out_f32 = 0) or
 // float32.  Needs 16-byte aligned bases and row strides (K % 8 == 0): else KL_ERR_BAD_ALIGN.  swiglu: 0 plain, 1 silu(gate) * up,
-// 2 gelu(gate) * up (see set_gated).
+// 2 gelu(gate) * up, 3 relu(gate) * up, 4 the clamped form with limit, alpha, shift (see set_gated).
 KL_API int kl_gemm_tcgen05(const void* a, long long lda, const void* w, long long ldw, void* out, long long ldo, int M,
-                           int N, int K, int out_f32, int swiglu, int* status, cudaStream_t stream) {
+                           int N, int K, int out_f32, int swiglu, float limit, float alpha, float shift, int* status, cudaStream_t stream) {
     if (M <= 0 || N <= 0) return KL_OK;
-    if (swiglu < 0 || swiglu > 2 || (swiglu && (out_f32 || N % 128))) return KL_ERR_BAD_SIZE;
+    if (swiglu < 0 || swiglu > GATED_KINDS || (swiglu && (out_f32 || N % 128))) return KL_ERR_BAD_SIZE;
     if (!aligned_operand(a, lda, K) || !aligned_operand(w, ldw, K)) return KL_ERR_BAD_ALIGN;
     CUtensorMap ma, mb;
     int rc;
@@ -754,13 +759,13 @@ KL_API int kl_gemm_tcgen05(const void* a, long long lda, const void* w, long lon
         const int tiles_m2 = (M + 2 * TC_BM - 1) / (2 * TC_BM), tiles_n2 = (N + 255) / 256;
         if ((long long)tiles_m2 * tiles_n2 > 0x3fffffffLL) return KL_ERR_BAD_SIZE;
         GemmArgs pargs{out, ldo, 0, M, N, (K + TC_BK - 1) / TC_BK, out_f32, status, tiles_m2, tiles_n2, swiglu};
-        set_gated(pargs, swiglu);
+        set_gated(pargs, swiglu, limit, alpha, shift);
         return launch_pairs(ma, mb, pargs, 2 * min(tiles_m2 * tiles_n2, sms2 / 2), stream);
     }
     if ((rc = make_map(&mb, w, N, K, ldw, 256)) != KL_OK) return rc;
     const int tiles_m = (M + TC_BM - 1) / TC_BM, tiles_n = (N + 255) / 256;
     GemmArgs args{out, ldo, 0, M, N, (K + TC_BK - 1) / TC_BK, out_f32, status, tiles_m, tiles_n, swiglu};
-    set_gated(args, swiglu);
+    set_gated(args, swiglu, limit, alpha, shift);
     if ((long long)tiles_m * tiles_n > 0x7fffffffLL) return KL_ERR_BAD_SIZE;
     const int sms = kl::sm_count();
     if (sms <= 0) return KL_ERR_SETUP;
@@ -843,13 +848,14 @@ KL_API int kl_gemm_tcgen05_grouped_skinny(const void* a, long long lda, const vo
 // rsqrt(sum / K + scale_eps): with activations x * w this is the product of the normalised rows,
 // norm(x) = w * x / rms(x).  Together they remove the add-and-normalise kernel between two products.
 KL_API int kl_gemm_tcgen05_skinny(const void* a, long long lda, const void* w, long long ldw, void* out, long long ldo,
-                                  int M, int N, int K, int splits, int out_f32, int swiglu, const float* scale_ss,
+                                  int M, int N, int K, int splits, int out_f32, int swiglu, float limit, float alpha, float shift,
+                                  const float* scale_ss,
                                   int scale_ss_n, float scale_eps, float* sink, float* sink_ss, int* sink_counters,
                                   const float* sink_w, void* sink_scaled, int* status, cudaStream_t stream) {
     if (M <= 0 || N <= 0) return KL_OK;
     if (M > 512) return KL_ERR_BAD_SIZE;
     if (M > 64 && (scale_ss != nullptr || sink != nullptr)) return KL_ERR_BAD_SIZE;     // the folded norm: one tile of tokens
-    if (swiglu < 0 || swiglu > 2 || (swiglu && (splits != 1 || out_f32 || N % 128))) return KL_ERR_BAD_SIZE;
+    if (swiglu < 0 || swiglu > GATED_KINDS || (swiglu && (splits != 1 || out_f32 || N % 128))) return KL_ERR_BAD_SIZE;
     if (!aligned_operand(w, ldw, K) || !aligned_operand(a, lda, K)) return KL_ERR_BAD_ALIGN;
     if (scale_ss != nullptr && scale_ss_n < 1) return KL_ERR_BAD_SIZE;
     if (sink != nullptr && (!out_f32 || swiglu || sink_ss == nullptr || sink_counters == nullptr || ldo != N ||
@@ -868,7 +874,7 @@ KL_API int kl_gemm_tcgen05_skinny(const void* a, long long lda, const void* w, l
     const int token_tiles = (M + bn - 1) / bn;
     GemmArgs args{out, ldo, (long long)M * ldo, N, M, k_blocks, out_f32, status, token_tiles, 0, swiglu,
                   scale_ss, scale_ss_n, scale_eps, K, sink, sink_ss, sink_counters, sink_w, (__nv_bfloat16*)sink_scaled};
-    set_gated(args, swiglu);
+    set_gated(args, swiglu, limit, alpha, shift);
     dim3 grid(((N + TC_BM - 1) / TC_BM) * token_tiles, 1, splits);
     // A grid of at most one CTA per SM (small matrices) gives each CTA the whole of the SM's shared
     // memory as stages: what a CTA has in flight bounds what it streams (96 KB over the 1.5 us a tile

@@ -3,14 +3,19 @@
 //   moe_route_kernel    a warp per token: s = softmax(z) over all experts in 32 bits (z plus a bias per expert
 //                       where one is given), the `top` largest (the lower index among equals), their scores
 //                       as weights (divided by their sum if asked, which is the softmax over the chosen
-//                       logits alone).  Or s = sigmoid(z), with a correction per expert that joins the scores for
-//                       the choice but not for the weights; weights times a scale.
+//                       logits alone).  Or s = sigmoid(z).  With either a correction per expert may join the scores
+//                       for the choice but not for the weights; weights times a scale.
 //   moe_plan_kernel     one CTA: counts per expert, a list of (token, choice) pairs sorted by expert in
 //                       which every expert's run is padded to whole tiles, the expert of every tile, and
-//                       each pair's place in the list.  Everything stays on the device, so a step with
-//                       experts needs no answer from the host and can be captured in a graph.
+//                       each pair's place in the list (-1: the row belongs to no sequence, -2: the choice is
+//                       an identity expert, one whose number is not below `experts`, which has no product).
+//                       Everything stays on the device, so a step with experts needs no answer from the host
+//                       and can be captured in a graph.
 //   moe_combine_kernel  out[t] = sum over the token's choices, in the order of the choices, of
-//                       weight * (the expert's result at the pair's place), in 32 bits.
+//                       weight * (the expert's result at the pair's place, or for an identity expert the
+//                       layer's input row), in 32 bits; optionally plus the result of an expert that every
+//                       token takes (rows, or float32 pieces of a product), times sigmoid(a number per token)
+//                       where one is given.
 //
 // The order of the pairs inside an expert's run is whatever the counters gave; no result depends on it,
 // because the grouped product computes every row by itself.  ExiledOfCode/KuiperLLama has dense
@@ -58,11 +63,18 @@ moe_route_kernel(const RouteArgs A) {
         w[i] = 0.f;
         if (e < experts) {
             w[i] = A.sigmoid ? 1.0f / (1.0f + expf(-s[i])) : expf(s[i] - m);
-            s[i] = A.correction ? w[i] + A.correction[e] : w[i];
+            s[i] = w[i];
             sum += w[i];
         }
     }
     sum = A.sigmoid ? 1.f : warp_sum(sum);                   // softmax: scores are w / sum
+    if (A.correction != nullptr) {
+#pragma unroll
+        for (int i = 0; i < MOE_MAX_PER_LANE; ++i) {
+            const int e = lane + 32 * i;
+            if (e < experts) s[i] = w[i] / sum + A.correction[e];
+        }
+    }
     float* weight = A.weight + (size_t)t * top;
     if (groups > 1 && A.keep_groups < groups) {
         // Experts form `groups` equal groups of neighbours; a group's score is its largest choice score, or the sum of its
@@ -155,7 +167,7 @@ moe_plan_kernel(const int* __restrict__ choice, const int* __restrict__ token_sl
     for (int p = threadIdx.x; p < pairs; p += blockDim.x) {
         const int t = p / top;
         const bool live = token_slot == nullptr || token_slot[t] >= 0;
-        rank[p] = live ? atomicAdd(&count[choice[p]], 1) : -1;
+        rank[p] = !live ? -1 : (choice[p] >= experts ? -2 : atomicAdd(&count[choice[p]], 1));
     }
     __syncthreads();
     if (threadIdx.x == 0) {
@@ -171,41 +183,41 @@ moe_plan_kernel(const int* __restrict__ choice, const int* __restrict__ token_sl
         for (int tile = first[e] / tile_rows; tile < first[e + 1] / tile_rows; ++tile) tile_group[tile] = e;
     for (int p = threadIdx.x; p < pairs; p += blockDim.x) {
         const int r = rank[p];
-        const int pos = r < 0 ? -1 : first[choice[p]] + r;
+        const int pos = r < 0 ? r : first[choice[p]] + r;
         pair_pos[p] = pos;
         if (pos >= 0) list_rows[pos] = p / top;
     }
 }
 
-template <typename T>
-__global__ void __launch_bounds__(256)
-moe_combine_kernel(const T* __restrict__ results, long long ld, const int* __restrict__ pair_pos, const float* __restrict__ weight,
-                   int tokens, int top, int hidden, float* __restrict__ out) {
-    pdl_launch_dependents();
-    pdl_wait();
-    const size_t total = (size_t)tokens * hidden;
-    for (size_t idx = (size_t)blockIdx.x * blockDim.x + threadIdx.x; idx < total; idx += (size_t)gridDim.x * blockDim.x) {
-        const size_t t = idx / hidden;
-        const int c = (int)(idx - t * hidden);
-        float acc = 0.f;
-        for (int k = 0; k < top; ++k) {
-            const int pos = pair_pos[t * top + k];
-            if (pos >= 0) acc = fmaf(weight[t * top + k], to_f32(results[(size_t)pos * ld + c]), acc);
-        }
-        out[idx] = acc;
+struct CombineArgs {
+    const void* results; long long ld;             // the list's rows, compute dtype
+    const int* pair_pos; const float* weight;
+    const void* x; long long x_ld;                 // the layer's input rows, compute dtype (identity experts), or null
+    const void* shared; long long shared_ld;       // the expert every token takes: rows in the compute dtype, or null
+    const float* pieces; int n_pieces; long long piece_stride;   // or float32 [n_pieces][tokens][hidden]
+    const float* gate; long long gate_ld;          // its factor is sigmoid(gate[t * gate_ld]); null: 1
+    int tokens, top, hidden;
+    float* out;
+};
+
+// V elements of a row a thread (V = 16 bytes of results an access where rows allow it, else 1), a token's results on their way four
+// at a time.
+template <typename T, int V> __device__ __forceinline__ void mc_load(const T* p, float (&x)[V]) {
+    if constexpr (V == 1) x[0] = to_f32(p[0]);
+    else {
+        const uint4 raw = *reinterpret_cast<const uint4*>(p);
+        const T* e = reinterpret_cast<const T*>(&raw);
+#pragma unroll
+        for (int i = 0; i < V; ++i) x[i] = to_f32(e[i]);
     }
 }
-
-// The same, V elements of a row a thread (16 bytes of results an access), a token's results on their way four at a time.
-template <typename T>
+template <typename T, int V>
 __global__ void __launch_bounds__(256)
-moe_combine_vec_kernel(const T* __restrict__ results, long long ld, const int* __restrict__ pair_pos, const float* __restrict__ weight,
-                       int tokens, int top, int hidden, float* __restrict__ out) {
+moe_combine_kernel(const CombineArgs A) {
     pdl_launch_dependents();
     pdl_wait();
-    constexpr int V = 16 / sizeof(T);
-    const int per = hidden / V;
-    const size_t total = (size_t)tokens * per;
+    const int per = A.hidden / V, top = A.top;
+    const size_t total = (size_t)A.tokens * per;
     for (size_t idx = (size_t)blockIdx.x * blockDim.x + threadIdx.x; idx < total; idx += (size_t)gridDim.x * blockDim.x) {
         const size_t t = idx / per;
         const int c = (int)(idx - t * per) * V;
@@ -213,24 +225,48 @@ moe_combine_vec_kernel(const T* __restrict__ results, long long ld, const int* _
 #pragma unroll
         for (int e = 0; e < V; ++e) acc[e] = 0.f;
         for (int k0 = 0; k0 < top; k0 += 4) {
-            uint4 raw[4];
-            float wt[4];
+            float r[4][V], wt[4];
 #pragma unroll
             for (int k = 0; k < 4; ++k) {
-                const int pos = k0 + k < top ? pair_pos[t * top + k0 + k] : -1;
-                wt[k] = pos >= 0 ? weight[t * top + k0 + k] : 0.f;
-                raw[k] = pos >= 0 ? *reinterpret_cast<const uint4*>(results + (size_t)pos * ld + c) : make_uint4(0u, 0u, 0u, 0u);
+                const int pos = k0 + k < top ? A.pair_pos[t * top + k0 + k] : -1;
+                const T* src = pos >= 0 ? (const T*)A.results + (size_t)pos * A.ld + c
+                                        : (pos == -2 && A.x != nullptr ? (const T*)A.x + t * A.x_ld + c : nullptr);
+                wt[k] = src != nullptr ? A.weight[t * top + k0 + k] : 0.f;
+                if (src != nullptr) mc_load<T, V>(src, r[k]);
+                else {
+#pragma unroll
+                    for (int e = 0; e < V; ++e) r[k][e] = 0.f;
+                }
             }
 #pragma unroll
-            for (int k = 0; k < 4; ++k) {
-                const T* p = reinterpret_cast<const T*>(&raw[k]);
+            for (int k = 0; k < 4; ++k)
 #pragma unroll
-                for (int e = 0; e < V; ++e) acc[e] = fmaf(wt[k], to_f32(p[e]), acc[e]);
-            }
+                for (int e = 0; e < V; ++e) acc[e] = fmaf(wt[k], r[k][e], acc[e]);
         }
-        float* o = out + t * hidden + c;
+        if (A.shared != nullptr || A.n_pieces > 0) {
+            float y[V];
 #pragma unroll
-        for (int e = 0; e < V; e += 4) *reinterpret_cast<float4*>(o + e) = make_float4(acc[e], acc[e + 1], acc[e + 2], acc[e + 3]);
+            for (int e = 0; e < V; ++e) y[e] = 0.f;
+            if (A.shared != nullptr) mc_load<T, V>((const T*)A.shared + t * A.shared_ld + c, y);
+            for (int z = 0; z < A.n_pieces; ++z) {
+                const float* p = A.pieces + (size_t)z * A.piece_stride + t * A.hidden + c;
+                if constexpr (V % 4 == 0) {
+#pragma unroll
+                    for (int e = 0; e < V; e += 4) {
+                        const float4 q = *reinterpret_cast<const float4*>(p + e);
+                        y[e] += q.x; y[e + 1] += q.y; y[e + 2] += q.z; y[e + 3] += q.w;
+                    }
+                } else y[0] += p[0];
+            }
+            const float f = A.gate != nullptr ? 1.0f / (1.0f + expf(-A.gate[t * A.gate_ld])) : 1.0f;
+#pragma unroll
+            for (int e = 0; e < V; ++e) acc[e] = fmaf(f, y[e], acc[e]);
+        }
+        float* o = A.out + t * A.hidden + c;
+        if constexpr (V % 4 == 0) {
+#pragma unroll
+            for (int e = 0; e < V; e += 4) *reinterpret_cast<float4*>(o + e) = make_float4(acc[e], acc[e + 1], acc[e + 2], acc[e + 3]);
+        } else o[0] = acc[0];
     }
 }
 
@@ -295,26 +331,26 @@ KL_API int kl_moe_plan(const int* choice, const int* token_slot, int tokens, int
     return KL_OK;
 }
 
-KL_API int kl_moe_combine(const void* results, long long ld, const int* pair_pos, const float* weight, int tokens, int top,
-                          int hidden, float* out, int dtype, cudaStream_t stream) {
+// x: the layer's input rows (compute dtype; needed where pair_pos has identity experts) or null.  The expert every token takes: rows
+// `shared` (compute dtype) or float32 pieces [n_pieces][tokens][hidden], or neither; gate: float32, the token's number at t * gate_ld, or null.
+KL_API int kl_moe_combine(const void* results, long long ld, const int* pair_pos, const float* weight, const void* x, long long x_ld,
+                          const void* shared, long long shared_ld, const float* pieces, int n_pieces, long long piece_stride,
+                          const float* gate, long long gate_ld, int tokens, int top, int hidden, float* out, int dtype, cudaStream_t stream) {
     if (tokens <= 0 || hidden <= 0) return KL_OK;
+    if (dtype != KL_F32 && dtype != KL_BF16) return KL_ERR_BAD_DTYPE;
+    if (n_pieces < 0 || (n_pieces > 0 && (pieces == nullptr || shared != nullptr))) return KL_ERR_BAD_SIZE;
+    const CombineArgs A{results, ld, pair_pos, weight, x, x_ld, shared, shared_ld, pieces, n_pieces, piece_stride, gate, gate_ld, tokens, top, hidden, out};
     const int v = dtype == KL_F32 ? 4 : 8;
-    if ((dtype == KL_F32 || dtype == KL_BF16) && hidden % v == 0 && ld % v == 0 && (((uintptr_t)results | (uintptr_t)out) & 15) == 0) {
-        const int grid = kl::strided_grid((size_t)tokens * (hidden / v), 256, 16);
-        if (dtype == KL_F32)
-            launch_kernel(moe_combine_vec_kernel<float>, grid, 256, 0, stream, (const float*)results, ld, pair_pos, weight, tokens, top, hidden, out);
-        else
-            launch_kernel(moe_combine_vec_kernel<bf16>, grid, 256, 0, stream, (const bf16*)results, ld, pair_pos, weight, tokens, top, hidden, out);
-        KL_LAUNCH_CHECK();
-        return KL_OK;
+    const bool wide = hidden % v == 0 && ld % v == 0 && x_ld % v == 0 && shared_ld % v == 0 && piece_stride % v == 0 &&
+                      (((uintptr_t)results | (uintptr_t)out | (uintptr_t)x | (uintptr_t)shared | (uintptr_t)pieces) & 15) == 0;
+    const int grid = kl::strided_grid((size_t)tokens * (wide ? hidden / v : hidden), 256, 16);
+    if (dtype == KL_F32) {
+        if (wide) launch_kernel(moe_combine_kernel<float, 4>, grid, 256, 0, stream, A);
+        else launch_kernel(moe_combine_kernel<float, 1>, grid, 256, 0, stream, A);
+    } else {
+        if (wide) launch_kernel(moe_combine_kernel<bf16, 8>, grid, 256, 0, stream, A);
+        else launch_kernel(moe_combine_kernel<bf16, 1>, grid, 256, 0, stream, A);
     }
-    const int blocks = kl::strided_grid((size_t)tokens * hidden, 256, 16);
-    if (dtype == KL_F32)
-        launch_kernel(moe_combine_kernel<float>, blocks, 256, 0, stream, (const float*)results, ld, pair_pos, weight, tokens, top, hidden, out);
-    else if (dtype == KL_BF16)
-        launch_kernel(moe_combine_kernel<bf16>, blocks, 256, 0, stream, (const bf16*)results, ld, pair_pos, weight, tokens, top, hidden, out);
-    else
-        return KL_ERR_BAD_DTYPE;
     KL_LAUNCH_CHECK();
     return KL_OK;
 }

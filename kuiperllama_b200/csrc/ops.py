@@ -104,19 +104,26 @@ def _i32(t: Optional[torch.Tensor], name: str) -> None:
 # --------------------------------------------------------------------------- row-wise
 
 def embedding(ids: torch.Tensor, table: torch.Tensor, out: torch.Tensor, error_flag: torch.Tensor,
-              scale: float = 1.0, positions: Optional[torch.Tensor] = None, freq: Optional[torch.Tensor] = None) -> None:
+              scale: float = 1.0, positions: Optional[torch.Tensor] = None, freq: Optional[torch.Tensor] = None,
+              position_table: Optional[torch.Tensor] = None) -> None:
     """out[t] = scale * float32(table[ids[t]]); ids outside the table set error_flag[0] = 1.  With ``freq`` (float32
     [2, ceil(hidden / 2)]: a frequency per pair, and what its rounding left over) a sinusoid of ``positions`` is added in the
-    same kernel: sin(p f_i) to entry 2i, cos(p f_i) to entry 2i + 1."""
-    _cuda(ids, table, out, error_flag, positions, freq)
+    same kernel: sin(p f_i) to entry 2i, cos(p f_i) to entry 2i + 1.  With ``position_table`` (a vector per position, in the
+    table's dtype) row ``positions[t]`` of it is added instead; a position outside it is flagged like an id."""
+    _cuda(ids, table, out, error_flag, positions, freq, position_table)
     _i32(ids, "ids"); _i32(error_flag, "error_flag"); _i32(positions, "positions")
     n, (vocab, hidden) = ids.numel(), table.shape
     _need(table.is_contiguous() and out.is_contiguous() and out.dtype == torch.float32, "embedding: bad layout")
     _need(out.shape[0] >= n and out.shape[1] == hidden, "embedding: output shape")
     _need(freq is None or (positions is not None and positions.numel() >= n and freq.dtype == torch.float32 and freq.is_contiguous()
                            and tuple(freq.shape) == (2, (hidden + 1) // 2)), "embedding: frequencies [2, pairs] and a position per token")
+    _need(position_table is None or (freq is None and positions is not None and positions.numel() >= n and position_table.dtype == table.dtype
+                                     and position_table.is_contiguous() and position_table.dim() == 2 and position_table.shape[1] == hidden),
+          "embedding: position vectors [positions, hidden] in the table's dtype and a position per token")
+    added = freq is not None or position_table is not None
     _check(lib("rowwise").kl_embedding(_ptr(ids), n, _ptr(table), dtype_code(table.dtype), vocab, hidden, ctypes.c_float(scale),
-                                       _ptr(positions if freq is not None else None), _ptr(freq), _ptr(out), _ptr(error_flag), _stream()), "embedding")
+                                       _ptr(positions if added else None), _ptr(freq), _ptr(position_table),
+                                       0 if position_table is None else position_table.shape[0], _ptr(out), _ptr(error_flag), _stream()), "embedding")
 
 
 def logit_transform(logits: torch.Tensor, scale: float = 1.0, softcap: float = 0.0) -> None:
@@ -164,16 +171,27 @@ def add_rmsnorm(residual: torch.Tensor, delta: Optional[torch.Tensor], weight: t
                                          dtype_code(out.dtype), _stream()), "add_rmsnorm")
 
 
-GATED_ACTIVATIONS = {"silu": 1, "gelu_tanh": 2}     # what a gated feed-forward applies to its gate
+GATED_ACTIVATIONS = {"silu": 1, "gelu_tanh": 2, "relu": 3}     # what a gated feed-forward applies to its gate
 
 
-def swiglu(gate_up: torch.Tensor, out: torch.Tensor, activation: str = "silu") -> None:
-    """out[t, i] = act(gate_up[t, i]) * gate_up[t, I + i], act one of ``GATED_ACTIVATIONS``."""
+def _gated_args(activation) -> tuple:
+    """The kernels' arguments for a gated activation: act(gate) * up by name (``GATED_ACTIVATIONS``), or (limit, alpha, shift):
+    min(g, limit) * sigmoid(alpha * min(g, limit)) * (clamp(u, -limit, limit) + shift), no clamp when limit <= 0."""
+    kind, form = (GATED_ACTIVATIONS[activation], (0.0, 1.0, 0.0)) if isinstance(activation, str) else (4, activation)
+    return (kind,) + tuple(ctypes.c_float(v) for v in form)
+
+
+_UNGATED = (0, ctypes.c_float(0.0), ctypes.c_float(1.0), ctypes.c_float(0.0))
+
+
+def swiglu(gate_up: torch.Tensor, out: torch.Tensor, activation="silu") -> None:
+    """out[t, i] = act(gate_up[t, i]) * gate_up[t, I + i], act one of ``GATED_ACTIVATIONS`` or a (limit, alpha, shift)
+    (``_gated_args``)."""
     _cuda(gate_up, out)
     tokens, two_i = gate_up.shape
     _need(two_i % 2 == 0 and out.shape == (tokens, two_i // 2), "swiglu: shapes")
     _need(gate_up.is_contiguous() and out.is_contiguous() and gate_up.dtype == out.dtype, "swiglu: layout")
-    _check(lib("rowwise").kl_swiglu(_ptr(gate_up), _ptr(out), tokens, two_i // 2, GATED_ACTIVATIONS[activation] - 1, dtype_code(out.dtype), _stream()),
+    _check(lib("rowwise").kl_swiglu(_ptr(gate_up), _ptr(out), tokens, two_i // 2, *_gated_args(activation), dtype_code(out.dtype), _stream()),
            "swiglu")
 
 
@@ -300,6 +318,46 @@ def pair_rmsnorm(residual: torch.Tensor, deltas, w1: Optional[torch.Tensor], w2:
               "pair_rmsnorm: output shape")
     _check(lib("norms").kl_pair_rmsnorm(_ptr(residual), *args, _ptr(w1), _ptr(w2), ctypes.c_float(eps), _ptr(out1), _ptr(out2), _ptr(rows),
                                         n, hidden, dtype_code(dtype), _stream()), "pair_rmsnorm")
+
+
+MAX_STREAMS = 16               # equals ST_MAX_STREAMS in streams.cu
+
+
+def stream_norm(streams: torch.Tensor, delta: Optional[torch.Tensor], out: Optional[torch.Tensor], weight: Optional[torch.Tensor], eps: float, *,
+                mix: Optional[torch.Tensor] = None, out_weights: Optional[torch.Tensor] = None, in_weights: Optional[torch.Tensor] = None,
+                write: Optional[torch.Tensor] = None, n_streams: Optional[int] = None, rows: Optional[torch.Tensor] = None,
+                dtype: Optional[torch.dtype] = None) -> None:
+    """Several residual streams: x'_t = sum_s mix[s, t] x_s + out_weights[t] * delta (without ``mix`` the streams stay), written to
+    ``write`` where given (float32 [rows, S, hidden], may be ``streams``); out = u / rms(u) * weight of u = sum_t in_weights[t] x'_t
+    (None: the plain sum).  ``streams``: float32 [rows, S, hidden], or [rows, hidden] with ``n_streams``: every stream is that row.
+    ``delta``: [rows, hidden] in the compute dtype (any row stride) or float32 pieces [P, rows, hidden].  ``out`` None: the
+    streams alone.  ``rows``: only those rows, nothing is written back."""
+    _cuda(streams, delta, out, weight, mix, out_weights, in_weights, write, rows)
+    _i32(rows, "rows")
+    one = streams.dim() == 2
+    S = int(n_streams) if one else streams.shape[1]
+    total, hidden = streams.shape[0], streams.shape[-1]
+    n = rows.numel() if rows is not None else total
+    _need(streams.dtype == torch.float32 and streams.is_contiguous() and 1 <= S <= MAX_STREAMS, f"stream_norm: float32 streams, up to {MAX_STREAMS}")
+    _need(write is None or (rows is None and write.dtype == torch.float32 and write.is_contiguous() and tuple(write.shape) == (total, S, hidden)
+                            and not (one and write.data_ptr() == streams.data_ptr())), "stream_norm: write")
+    f32 = lambda t, size: t is None or (t.dtype == torch.float32 and t.is_contiguous() and t.numel() == size)
+    _need(f32(mix, S * S) and f32(out_weights, S) and f32(in_weights, S) and f32(weight, hidden), "stream_norm: float32 weights")
+    _need(out is None or (weight is not None and out.is_contiguous() and out.shape[0] >= n and out.shape[1] == hidden), "stream_norm: out")
+    if dtype is None:
+        dtype = out.dtype if out is not None else (delta.dtype if delta is not None and delta.dim() == 2 else torch.float32)
+    plain, parts, n_parts, stride = delta, None, 0, 0
+    if _partials(delta):
+        _need(delta.dtype == torch.float32 and delta.is_contiguous() and tuple(delta.shape[1:]) == (total, hidden),
+              "stream_norm: pieces must be float32 [P, rows, hidden]")
+        plain, parts, n_parts, stride = None, delta, delta.shape[0], delta.shape[1] * delta.shape[2]
+    elif delta is not None:
+        _need(delta.dtype == dtype and delta.dim() == 2 and delta.stride(1) == 1 and delta.shape[0] >= total and delta.shape[1] == hidden,
+              "stream_norm: delta must be [rows, hidden] in the compute dtype")
+    _check(lib("streams").kl_stream_norm(
+        _ptr(streams), ctypes.c_longlong(0 if one else hidden), ctypes.c_longlong(hidden if one else S * hidden), _ptr(write), _ptr(plain),
+        ctypes.c_longlong(0 if plain is None else plain.stride(0)), _ptr(parts), n_parts, ctypes.c_longlong(stride), _ptr(mix), _ptr(out_weights),
+        _ptr(in_weights), _ptr(weight), ctypes.c_float(eps), _ptr(out), _ptr(rows), n, S, hidden, dtype_code(dtype), _stream()), "stream_norm")
 
 
 def activation(x: torch.Tensor, out: torch.Tensor, kind: str, params: Optional[torch.Tensor] = None) -> None:
@@ -539,6 +597,60 @@ def qk_prepare(proj: torch.Tensor, q_col: int, k_col: int, v_col: Optional[int],
         _ptr(k_cache), _ptr(v_cache), n_tokens, H, KV, hd, vd, dtype_code(proj.dtype), _stream()), "qk_prepare")
 
 
+QKV_CONV_MAX_TAPS = 16         # equals QC_MAX_TAPS in qkv_conv.cu
+
+
+def qkv_conv(proj: torch.Tensor, q_col: int, k_col: int, v_col: int, q_out: torch.Tensor, step, block_table: Optional[torch.Tensor],
+             k_cache: Optional[torch.Tensor], v_cache: Optional[torch.Tensor], num_heads: int, num_kv_heads: int, head_dim: int,
+             value_dim: int, *, conv_weight: Optional[torch.Tensor] = None, state: Optional[torch.Tensor] = None,
+             inv_freq: Optional[torch.Tensor] = None, rotary_dim: int = 0, magnitude: float = 1.0, interleaved: bool = False,
+             v_first: Optional[torch.Tensor] = None, v_lambda: Optional[torch.Tensor] = None, v_keep: Optional[torch.Tensor] = None) -> None:
+    """Per token, in one kernel: a short causal convolution on every channel of the projected q, k and v (``conv_weight``
+    float32 [taps, width of proj], by column of ``proj``; None: none), the rotation of the first ``rotary_dim`` elements of every q
+    and k head (cos and sin times ``magnitude``), value mixing as in ``qk_row_prepare`` (``v_keep`` gets the values behind the
+    convolution), q into ``q_out``, k and v into the cache.  ``state`` float32 [slots, >= (taps - 1) * width]: the sequences' last
+    taps - 1 rows of ``proj``, oldest first; it moves on.  ``proj``: [rows, width] in ``q_out``'s dtype, or, in a step of one
+    token per sequence, float32 pieces [S, rows, width] of the product."""
+    _cuda(proj, q_out, block_table, k_cache, v_cache, conv_weight, state, inv_freq, v_first, v_lambda, v_keep)
+    H, KV, hd, vd, n = num_heads, num_kv_heads, head_dim, value_dim, step.n_tokens
+    pieces = proj.dim() == 3
+    single = bool(step.is_decode)
+    _need(proj.stride(-1) == 1 and proj.shape[-2] >= n and (proj.dtype == torch.float32 and proj.is_contiguous() and single if pieces else proj.dtype == q_out.dtype),
+          "qkv_conv: rows in the compute dtype, or (one token per sequence) float32 pieces")
+    ld = proj.stride(-2)
+    for col, heads, size in ((q_col, H, hd), (k_col, KV, hd), (v_col, KV, vd)):
+        _need(col >= 0 and col + heads * size <= proj.shape[-1], "qkv_conv: projection columns")
+    taps = 1
+    if conv_weight is not None:
+        taps = conv_weight.shape[0]
+        _need(conv_weight.dtype == torch.float32 and conv_weight.is_contiguous() and 1 <= taps <= QKV_CONV_MAX_TAPS and conv_weight.shape[1] == ld == proj.shape[-1],
+              f"qkv_conv: weights float32 [taps (up to {QKV_CONV_MAX_TAPS}), width of the product]")
+    if taps > 1:
+        _need(state is not None and state.dtype == torch.float32 and state.dim() == 2 and state.stride(1) == 1 and state.shape[1] >= (taps - 1) * ld, "qkv_conv: state")
+    _need(rotary_dim == 0 or (inv_freq is not None and inv_freq.dtype == torch.float32 and inv_freq.is_contiguous() and 2 * inv_freq.numel() >= rotary_dim
+                              and rotary_dim <= hd and rotary_dim % 2 == 0), "qkv_conv: rotation")
+    _need(q_out.dim() == 2 and q_out.shape[0] >= n and q_out.shape[1] == H * hd and q_out.stride(1) == 1, "qkv_conv: q_out")
+    for c, size in ((k_cache, hd), (v_cache, vd)):
+        _need(c is None or (c.is_contiguous() and c.dtype == q_out.dtype and tuple(c.shape[1:]) == (KV, PAGE, size)), "qkv_conv: cache layout")
+    _need(v_first is None or (v_first.dtype == q_out.dtype and v_first.dim() == 2 and v_first.stride(1) == 1 and v_first.shape[0] >= n and v_first.shape[1] == KV * vd
+                              and v_lambda is not None and v_lambda.dtype == torch.float32), "qkv_conv: the values to mix in")
+    _need(v_keep is None or (v_keep.dtype == q_out.dtype and v_keep.is_contiguous() and v_keep.shape[0] >= n and v_keep.shape[1] == KV * vd), "qkv_conv: v_keep")
+    _i32(block_table, "block_table")
+    max_new = 1 if single else int(step.max_new)
+    _check(lib("qkv_conv").kl_qkv_conv(
+        _ptr(None if pieces else proj), _ptr(proj if pieces else None), proj.shape[0] if pieces else 0,
+        ctypes.c_longlong(proj.stride(0) if pieces else 0), ctypes.c_longlong(ld), q_col, k_col, v_col, _ptr(conv_weight), taps, _ptr(state),
+        ctypes.c_longlong(0 if state is None else state.stride(0)), _ptr(inv_freq), int(rotary_dim), int(bool(interleaved)), ctypes.c_float(magnitude),
+        _ptr(q_out), ctypes.c_longlong(q_out.stride(0)), _ptr(k_cache), _ptr(v_cache), _ptr(block_table),
+        0 if block_table is None else block_table.shape[1], _ptr(v_first), ctypes.c_longlong(0 if v_first is None else v_first.stride(0)),
+        _ptr(v_lambda), _ptr(v_keep), _ptr(step.cu_tokens), _ptr(step.seq_slots), _ptr(step.seq_starts), step.n_seqs, max_new, int(single),
+        H, KV, hd, vd, dtype_code(q_out.dtype), _stream()), "qkv_conv")
+    if taps > 1 and not single:
+        _check(lib("short_conv").kl_short_conv_state(
+            _ptr(proj), ctypes.c_longlong(ld), taps, _ptr(state), ctypes.c_longlong(state.stride(0)), _ptr(step.cu_tokens), _ptr(step.seq_slots),
+            step.n_seqs, ld, dtype_code(proj.dtype), _stream()), "short_conv_state")
+
+
 ATTENTION_WEIGHTS = {"softmax": 0, "sigmoid": 1}
 
 
@@ -705,14 +817,13 @@ def moe_route(logits: torch.Tensor, top: int, renormalise: bool = False, groups:
     softmax over all experts, the ``top`` largest, their scores (divided by their sum + ``renorm_eps`` if ``renormalise``).
     With ``groups`` > 1 the experts form that many equal groups of neighbours, a group's score is its largest score, and
     only experts of the ``keep_groups`` best groups can be chosen.  ``bias``: float32 [experts], added to the logits first.
-    ``scores`` "sigmoid": every expert's score is sigmoid(z) by itself; ``correction`` (float32 [experts]) joins the scores for
+    ``scores`` "sigmoid": every expert's score is sigmoid(z) by itself; ``correction`` (float32 [experts]) joins the (normalised) scores for
     the choice, of groups and experts alike, but not for the weights; ``group_top``: a group's score is the sum of its so many
     best; ``scale`` multiplies the weights."""
     _cuda(logits, bias, correction)
     _need(scores in ROUTER_SCORES, f"moe_route: scores {scores!r} ({', '.join(ROUTER_SCORES)})")
     _need(correction is None or (correction.dtype == torch.float32 and correction.is_contiguous() and correction.numel() == logits.shape[1]),
           "moe_route: float32 correction per expert")
-    _need(correction is None or scores == "sigmoid", "moe_route: a correction goes with sigmoid scores")
     _need(group_top >= 1, "moe_route: a group's score takes at least one expert")
     n, E = logits.shape
     _need(bias is None or (bias.dtype == torch.float32 and bias.is_contiguous() and bias.numel() == E), "moe_route: float32 bias per expert")
@@ -730,7 +841,8 @@ def moe_route(logits: torch.Tensor, top: int, renormalise: bool = False, groups:
 
 def moe_plan(choice: torch.Tensor, experts: int, tile_rows: int, token_slot: Optional[torch.Tensor] = None):
     """The list of (token, choice) pairs sorted by expert, every expert's run padded to whole tiles:
-    (pair_pos int32 [tokens * top]: each pair's place, -1 for rows that belong to no sequence; list_rows int32
+    (pair_pos int32 [tokens * top]: each pair's place, -1 for rows that belong to no sequence, -2 for a choice that is not
+    below ``experts`` (an identity expert: no product); list_rows int32
     [cap]: the token row of every place, -1 for padding; tile_group int32 [cap / tile_rows]: the expert of every tile)."""
     _cuda(choice, token_slot)
     _i32(choice, "choice"); _i32(token_slot, "token_slot")
@@ -795,14 +907,31 @@ def gemm_tcgen05_grouped_skinny(a: torch.Tensor, w: torch.Tensor, out: torch.Ten
         _epilogue_activation(activation, gated), _status_ptr(a.device), _stream()), "gemm_tcgen05_grouped_skinny")
 
 
-def moe_combine(results: torch.Tensor, pair_pos: torch.Tensor, weight: torch.Tensor, out: torch.Tensor) -> None:
-    """out[t] = sum_k weight[t, k] * results[pair_pos[t * top + k]] (float32 [tokens, hidden]), in the order of k."""
-    _cuda(results, pair_pos, weight, out)
+def moe_combine(results: torch.Tensor, pair_pos: torch.Tensor, weight: torch.Tensor, out: torch.Tensor, x: Optional[torch.Tensor] = None,
+                shared: Optional[torch.Tensor] = None, shared_gate: Optional[torch.Tensor] = None) -> None:
+    """out[t] = sum_k weight[t, k] * results[pair_pos[t * top + k]] (float32 [tokens, hidden]), in the order of k; where pair_pos
+    is -2 the term is weight[t, k] * x[t] (``x``: the layer's input rows).  ``shared``: the result of an expert that every token
+    takes, [tokens, hidden] in the results' dtype or float32 pieces [S, tokens, hidden], is added, times
+    sigmoid(shared_gate[t]) where ``shared_gate`` (float32 [tokens], any stride) is given."""
+    _cuda(results, pair_pos, weight, out, x, shared, shared_gate)
     n, top = weight.shape
     _need(out.dtype == torch.float32 and out.is_contiguous() and out.shape[0] >= n and results.stride(1) == 1
           and results.shape[1] == out.shape[1], "moe_combine: shapes")
-    _check(lib("moe").kl_moe_combine(_ptr(results), ctypes.c_longlong(results.stride(0)), _ptr(pair_pos), _ptr(weight), n, top,
-                                     out.shape[1], _ptr(out), dtype_code(results.dtype), _stream()), "moe_combine")
+    hidden = out.shape[1]
+    _need(x is None or (x.dtype == results.dtype and x.stride(1) == 1 and x.shape[0] >= n and x.shape[1] == hidden), "moe_combine: x")
+    rows, pieces, n_pieces, stride = shared, None, 0, 0
+    if shared is not None and shared.dim() == 3:
+        _need(shared.dtype == torch.float32 and shared.is_contiguous() and shared.shape[1] >= n and shared.shape[2] == hidden,
+              "moe_combine: shared pieces must be float32 [S, tokens, hidden]")
+        rows, pieces, n_pieces, stride = None, shared, shared.shape[0], shared.shape[1] * shared.shape[2]
+    elif shared is not None:
+        _need(shared.dtype == results.dtype and shared.stride(1) == 1 and shared.shape[0] >= n and shared.shape[1] == hidden, "moe_combine: shared rows")
+    _need(shared_gate is None or (shared_gate.dtype == torch.float32 and shared_gate.dim() == 1 and shared_gate.numel() >= n), "moe_combine: shared_gate")
+    _check(lib("moe").kl_moe_combine(
+        _ptr(results), ctypes.c_longlong(results.stride(0)), _ptr(pair_pos), _ptr(weight), _ptr(x), ctypes.c_longlong(0 if x is None else x.stride(0)),
+        _ptr(rows), ctypes.c_longlong(0 if rows is None else rows.stride(0)), _ptr(pieces), n_pieces, ctypes.c_longlong(stride),
+        _ptr(shared_gate), ctypes.c_longlong(0 if shared_gate is None else shared_gate.stride(0)), n, top, hidden, _ptr(out),
+        dtype_code(results.dtype), _stream()), "moe_combine")
 
 
 # --------------------------------------------------------------------------- attention over a shared latent
@@ -1323,11 +1452,11 @@ def skinny_splits(N: int, K: int, M: int = 1) -> int:
     return (k_blocks + per - 1) // per
 
 
-def gemm_tcgen05(a: torch.Tensor, w: torch.Tensor, out: torch.Tensor, swiglu: bool = False, activation: str = "silu") -> None:
+def gemm_tcgen05(a: torch.Tensor, w: torch.Tensor, out: torch.Tensor, swiglu: bool = False, activation="silu") -> None:
     """out[M, N] = a @ w^T on the tensor cores, tokens as tile rows (any M; pairs of CTAs on tiles of
     256 tokens where the token count suits, single CTAs on tiles of 128 otherwise).  With ``swiglu``
     the rows of ``w`` alternate 64 gate rows and 64 up rows and out[M, N / 2] receives
-    act(gate) * up (``activation`` one of ``GATED_ACTIVATIONS``)."""
+    act(gate) * up (``activation`` one of ``GATED_ACTIVATIONS``, or a (limit, alpha, shift))."""
     _cuda(a, w, out)
     (M, K), (N, K2) = a.shape, w.shape
     _need(K == K2 and out.shape[0] >= M and out.shape[1] == (N // 2 if swiglu else N), "gemm_tcgen05: shapes")
@@ -1335,7 +1464,7 @@ def gemm_tcgen05(a: torch.Tensor, w: torch.Tensor, out: torch.Tensor, swiglu: bo
     _need(_tc_ok(a, w, out), "gemm_tcgen05: operands must be bfloat16 with 16-byte aligned rows")
     _check(lib("gemm_tcgen05").kl_gemm_tcgen05(_ptr(a), ctypes.c_longlong(a.stride(0)), _ptr(w),
                                                ctypes.c_longlong(w.stride(0)), _ptr(out), ctypes.c_longlong(out.stride(0)),
-                                               M, N, K, int(out.dtype == torch.float32), GATED_ACTIVATIONS[activation] if swiglu else 0,
+                                               M, N, K, int(out.dtype == torch.float32), *(_gated_args(activation) if swiglu else _UNGATED),
                                                _status_ptr(a.device), _stream()), "gemm_tcgen05")
 
 
@@ -1387,7 +1516,7 @@ def gemm_skinny_stream(w: torch.Tensor, a: torch.Tensor, row_scale=None, sink=No
         _need(sink is None and N % 128 == 0, "gemm_skinny_stream: swiglu")
         out = torch.empty((M, N // 2), dtype=torch.bfloat16, device=dev)
         _check(L.kl_gemm_tcgen05_skinny(_ptr(a), ctypes.c_longlong(a.stride(0)), _ptr(w), ctypes.c_longlong(w.stride(0)), _ptr(out),
-                                        ctypes.c_longlong(out.stride(0)), M, N, K, 1, 0, 1, *scale_args, null, null, null, null,
+                                        ctypes.c_longlong(out.stride(0)), M, N, K, 1, 0, *_gated_args("silu"), *scale_args, null, null, null, null,
                                         null, st, _stream()), "gemm_skinny_stream")
         return out
     splits = skinny_splits(N, K, M) if splits is None else splits
@@ -1409,7 +1538,7 @@ def gemm_skinny_stream(w: torch.Tensor, a: torch.Tensor, row_scale=None, sink=No
                      _ptr(next_w) if next_w is not None else null, _ptr(scaled) if scaled is not None else null)
         result = (ss_out, scaled)
     _check(L.kl_gemm_tcgen05_skinny(_ptr(a), ctypes.c_longlong(a.stride(0)), _ptr(w), ctypes.c_longlong(w.stride(0)), _ptr(partial),
-                                    ctypes.c_longlong(N), M, N, K, splits, 1, 0, *scale_args, *sink_args, st, _stream()),
+                                    ctypes.c_longlong(N), M, N, K, splits, 1, *_UNGATED, *scale_args, *sink_args, st, _stream()),
            "gemm_skinny_stream")
     return result
 
@@ -1458,17 +1587,17 @@ def gemm_skinny_partials(a: torch.Tensor, w: torch.Tensor, splits: Optional[int]
     partial = torch.empty((splits, M, N), dtype=torch.float32, device=a.device)
     _check(lib("gemm_tcgen05").kl_gemm_tcgen05_skinny(
         _ptr(a), ctypes.c_longlong(a.stride(0)), _ptr(w), ctypes.c_longlong(w.stride(0)), _ptr(partial),
-        ctypes.c_longlong(N), M, N, K, splits, 1, 0, *_NO_STREAM_FUSION, _status_ptr(a.device), _stream()),
+        ctypes.c_longlong(N), M, N, K, splits, 1, *_UNGATED, *_NO_STREAM_FUSION, _status_ptr(a.device), _stream()),
         "gemm_skinny")
     return partial
 
 
 def gemm_skinny(a: torch.Tensor, w: torch.Tensor, out: torch.Tensor, splits: Optional[int] = None,
-                swiglu: bool = False, activation: str = "silu") -> None:
+                swiglu: bool = False, activation="silu") -> None:
     """out[M, N] = a @ w^T for M <= SKINNY_MAX_ROWS tokens: weights as tile rows, each weight read once, the
     K range cut into ``splits`` pieces whose float32 partial sums are added in a fixed order.
     With ``swiglu`` (rows of ``w`` alternate 64 gate and 64 up rows; no cut) out[M, N / 2]
-    receives act(gate) * up (``activation`` one of ``GATED_ACTIVATIONS``)."""
+    receives act(gate) * up (``activation`` one of ``GATED_ACTIVATIONS``, or a (limit, alpha, shift))."""
     _cuda(a, w, out)
     (M, K), (N, K2) = a.shape, w.shape
     _need(K == K2 and out.shape[0] >= M and out.shape[1] == (N // 2 if swiglu else N) and M <= SKINNY_MAX_ROWS, "gemm_skinny: shapes")
@@ -1480,12 +1609,12 @@ def gemm_skinny(a: torch.Tensor, w: torch.Tensor, out: torch.Tensor, splits: Opt
     if splits == 1:
         _check(L.kl_gemm_tcgen05_skinny(_ptr(a), ctypes.c_longlong(a.stride(0)), _ptr(w), ctypes.c_longlong(w.stride(0)),
                                         _ptr(out), ctypes.c_longlong(out.stride(0)), M, N, K, 1,
-                                        int(out.dtype == torch.float32), GATED_ACTIVATIONS[activation] if swiglu else 0,
+                                        int(out.dtype == torch.float32), *(_gated_args(activation) if swiglu else _UNGATED),
                                         *_NO_STREAM_FUSION, st, _stream()), "gemm_skinny")
         return
     partial = torch.empty((splits, M, N), dtype=torch.float32, device=a.device)
     _check(L.kl_gemm_tcgen05_skinny(_ptr(a), ctypes.c_longlong(a.stride(0)), _ptr(w), ctypes.c_longlong(w.stride(0)),
-                                    _ptr(partial), ctypes.c_longlong(N), M, N, K, splits, 1, 0, *_NO_STREAM_FUSION, st,
+                                    _ptr(partial), ctypes.c_longlong(N), M, N, K, splits, 1, *_UNGATED, *_NO_STREAM_FUSION, st,
                                     _stream()), "gemm_skinny")
     _check(L.kl_splitk_reduce(_ptr(partial), splits, M, N, _ptr(out), ctypes.c_longlong(out.stride(0)),
                               int(out.dtype == torch.float32), _stream()), "splitk_reduce")
@@ -1595,18 +1724,19 @@ def attention_mma(q: torch.Tensor, q_stride: int, out: torch.Tensor, k_cache: to
         "attention_mma", 2 if splits > 1 else 1)
 
 
-CHUNKED_MMA_DIMS = (32, 64, 128)       # key and value sizes of the tensor-core kernel with chunks and a distance bias
+CHUNKED_MMA_DIMS = (32, 64, 96, 128)   # key and value sizes of the tensor-core kernel with values of their own size
 
 
 def attention_chunked_mma(q: torch.Tensor, q_stride: int, out: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Tensor,
                           block_table: torch.Tensor, step, num_heads: int, num_kv_heads: int, head_dim: int, value_dim: int, scale: float,
-                          *, window: int = 0, chunk: int = 0, distance_bias: Optional[torch.Tensor] = None, splits: int = 1,
-                          few_rows: bool = False) -> None:
+                          *, window: int = 0, chunk: int = 0, distance_bias: Optional[torch.Tensor] = None, sink: Optional[torch.Tensor] = None,
+                          splits: int = 1, few_rows: bool = False) -> None:
     """Tensor-core softmax attention of ``step`` over the keys of every token's own chunk of ``chunk`` positions (0: no chunks;
     a ``window`` may cut them further), with ``distance_bias`` (float32 [heads, n]: column min(distance, n - 1) joins the
-    scaled score) and values of ``value_dim`` columns; bfloat16, key and value sizes of 32, 64 and 128, groups of up to 16 heads.
-    ``few_rows`` and ``splits`` as for ``attention_mma``."""
-    _cuda(q, out, k_cache, v_cache, block_table, distance_bias)
+    scaled score), a ``sink`` (float32 [heads]: exp(sink) joins the softmax's denominator) and values of ``value_dim`` columns;
+    bfloat16, key and value sizes of 32, 64, 96 and 128, groups of up to 16 heads.  ``few_rows`` and ``splits`` as for ``attention_mma``."""
+    _cuda(q, out, k_cache, v_cache, block_table, distance_bias, sink)
+    _need(sink is None or (sink.dtype == torch.float32 and sink.is_contiguous() and sink.numel() == num_heads), "attention_chunked_mma: sink")
     _i32(block_table, "block_table")
     H, KV, hd, vd, n = num_heads, num_kv_heads, head_dim, value_dim, step.n_tokens
     _need(q.dtype == out.dtype == k_cache.dtype == v_cache.dtype == torch.bfloat16, "attention_chunked_mma: bfloat16 only")
@@ -1620,11 +1750,11 @@ def attention_chunked_mma(q: torch.Tensor, q_stride: int, out: torch.Tensor, k_c
     if splits > 1:
         po = torch.empty((n, H, splits, vd), dtype=torch.float32, device=q.device)
         pml = torch.empty((n, H, splits, 2), dtype=torch.float32, device=q.device)
-    _check(lib("attention_mma").kl_attention_mma_chunked(
+    _check(lib("attention_mma_values").kl_attention_mma_chunked(
         _ptr(q), q_stride, _ptr(out), _ptr(k_cache), _ptr(v_cache), _ptr(block_table), block_table.shape[1], _ptr(step.cu_tokens),
         _ptr(step.seq_slots), _ptr(step.seq_starts), _ptr(step.seq_new), _ptr(po), _ptr(pml), step.n_seqs, int(step.max_new), n, H, KV, hd, vd,
         ctypes.c_float(scale), int(window or 0), splits, int(few_rows), int(chunk or 0), _ptr(distance_bias),
-        0 if distance_bias is None else distance_bias.shape[1], _stream()), "attention_chunked_mma", 2 if splits > 1 else 1)
+        0 if distance_bias is None else distance_bias.shape[1], _ptr(sink), _stream()), "attention_chunked_mma", 2 if splits > 1 else 1)
 
 
 def swiglu_fusable(hidden: int, inter: int, dtype: torch.dtype) -> bool:
@@ -1640,7 +1770,7 @@ def interleave_gate_up(gate: torch.Tensor, up: torch.Tensor) -> torch.Tensor:
     return torch.stack([gate.view(inter // 64, 64, k), up.view(inter // 64, 64, k)], dim=1).reshape(2 * inter, k).contiguous()
 
 
-def matmul_swiglu(a: torch.Tensor, w_gate_up: torch.Tensor, out: torch.Tensor, activation: str = "silu") -> None:
+def matmul_swiglu(a: torch.Tensor, w_gate_up: torch.Tensor, out: torch.Tensor, activation="silu") -> None:
     """out[M, I] = act(a @ gate^T) * (a @ up^T) in one kernel; ``w_gate_up`` from ``interleave_gate_up``."""
     if weights_as_rows(a.shape[0], w_gate_up.shape[0], swiglu=True):
         gemm_skinny(a, w_gate_up, out, swiglu=True, activation=activation)

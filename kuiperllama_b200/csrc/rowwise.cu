@@ -16,17 +16,19 @@ namespace kl {
 // emb_kernel.cu:11-13).  With `freq` (float32 [2, ceil(hidden / 2)]: every pair's frequency and what its rounding to float32
 // left over) a sinusoid of the token's position is added: entry 2i gets sin(p f_i), entry 2i + 1 cos(p f_i).  The angle
 // is a 32-bit product; what it leaves out of the exact one (its rounding and the frequency's, 1e-4 at position 2,000, 5e-3 at
-// 100,000) comes in as a second-order correction.
+// 100,000) comes in as a second-order correction.  With `pos_table` (a learned vector per position, [pos_rows, hidden] in the
+// table's dtype) the token's row of it is added, unscaled; a position outside it is treated like a bad id.
 template <typename T>
 __global__ void embedding_kernel(const int* __restrict__ ids, const T* __restrict__ table, float* __restrict__ out,
                                  int hidden, int vocab, float scale, const int* __restrict__ positions, const float* __restrict__ freq,
-                                 int* __restrict__ error_flag) {
+                                 const T* __restrict__ pos_table, int pos_rows, int* __restrict__ error_flag) {
     pdl_launch_dependents();
     pdl_wait();
     const int t = blockIdx.x;
     const int id = ids[t];
     float* o = out + (size_t)t * hidden;
-    if (id < 0 || id >= vocab) {
+    const int at = pos_table != nullptr ? positions[t] : 0;
+    if (id < 0 || id >= vocab || (pos_table != nullptr && (at < 0 || at >= pos_rows))) {
         if (threadIdx.x == 0) atomicExch(error_flag, 1);
         for (int i = threadIdx.x; i < hidden; i += blockDim.x) o[i] = 0.f;
         return;
@@ -44,6 +46,11 @@ __global__ void embedding_kernel(const int* __restrict__ ids, const T* __restric
             o[2 * i] = fmaf(scale, to_f32(row[2 * i]), fmaf(rest, cs, fmaf(-half, sn, sn)));
             if (2 * i + 1 < hidden) o[2 * i + 1] = fmaf(scale, to_f32(row[2 * i + 1]), fmaf(-rest, sn, fmaf(-half, cs, cs)));
         }
+        return;
+    }
+    if (pos_table != nullptr) {
+        const T* learned = pos_table + (size_t)at * hidden;
+        for (int i = threadIdx.x; i < hidden; i += blockDim.x) o[i] = fmaf(scale, to_f32(row[i]), to_f32(learned[i]));
         return;
     }
     for (int i = threadIdx.x; i < hidden; i += blockDim.x) o[i] = scale * to_f32(row[i]);
@@ -186,19 +193,26 @@ add_rmsnorm_kernel(float* __restrict__ residual, const T* __restrict__ delta, co
     }
 }
 
-// out[t, i] = act(gu[t, i]) * gu[t, inter + i]; gu is [tokens, 2 * inter] (gate columns first); act = silu, or with
-// gelu the tanh form of gelu.
+// out[t, i] = act(gu[t, i]) * gu[t, inter + i]; gu is [tokens, 2 * inter] (gate columns first); act by kind: 1 silu, 2 the
+// tanh form of gelu, 3 relu; 4: min(g, limit) * sigmoid(alpha * min(g, limit)) * (clamp(u, -limit, limit) + shift), no clamp
+// when limit <= 0.
 template <typename T>
-__global__ void swiglu_kernel(const T* __restrict__ gu, T* __restrict__ out, int tokens, int inter, int gelu) {
+__global__ void swiglu_kernel(const T* __restrict__ gu, T* __restrict__ out, int tokens, int inter, int kind, float limit, float alpha, float shift) {
     pdl_launch_dependents();
     pdl_wait();
     const size_t n = (size_t)tokens * inter;
     for (size_t idx = (size_t)blockIdx.x * blockDim.x + threadIdx.x; idx < n; idx += (size_t)gridDim.x * blockDim.x) {
         const size_t t = idx / inter;
         const int i = (int)(idx - t * inter);
-        const float g = to_f32(gu[t * 2 * inter + i]);
-        const float u = to_f32(gu[t * 2 * inter + inter + i]);
-        const float a = gelu ? 0.5f * g * (1.0f + tanhf(0.7978845608028654f * (g + 0.044715f * g * g * g))) : g * (1.0f / (1.0f + expf(-g)));
+        float g = to_f32(gu[t * 2 * inter + i]);
+        float u = to_f32(gu[t * 2 * inter + inter + i]);
+        float a;
+        if (kind == 4) {
+            if (limit > 0.f) { g = fminf(g, limit); u = fminf(fmaxf(u, -limit), limit); }
+            a = g * (1.0f / (1.0f + expf(-alpha * g)));
+            u += shift;
+        } else if (kind == 3) a = fmaxf(g, 0.f);
+        else a = kind == 2 ? 0.5f * g * (1.0f + tanhf(0.7978845608028654f * (g + 0.044715f * g * g * g))) : g * (1.0f / (1.0f + expf(-g)));
         out[idx] = from_f32<T>(a * u);
     }
 }
@@ -232,14 +246,16 @@ KL_API int kl_logit_transform(float* logits, long long ld, int rows, int vocab, 
 }
 
 KL_API int kl_embedding(const int* ids, int n_tokens, const void* table, int table_dtype, int vocab, int hidden,
-                        float scale, const int* positions, const float* freq, float* out, int* error_flag, cudaStream_t stream) {
+                        float scale, const int* positions, const float* freq, const void* pos_table, int pos_rows, float* out,
+                        int* error_flag, cudaStream_t stream) {
     if (n_tokens <= 0) return KL_OK;
-    if (freq != nullptr && positions == nullptr) return KL_ERR_BAD_SIZE;
+    if ((freq != nullptr || pos_table != nullptr) && positions == nullptr) return KL_ERR_BAD_SIZE;
+    if (freq != nullptr && pos_table != nullptr) return KL_ERR_BAD_SIZE;
     const int threads = hidden >= 1024 ? 256 : 128;
     if (table_dtype == KL_F32)
-        launch_kernel(embedding_kernel<float>, n_tokens, threads, 0, stream, ids, (const float*)table, out, hidden, vocab, scale, positions, freq, error_flag);
+        launch_kernel(embedding_kernel<float>, n_tokens, threads, 0, stream, ids, (const float*)table, out, hidden, vocab, scale, positions, freq, (const float*)pos_table, pos_rows, error_flag);
     else if (table_dtype == KL_BF16)
-        launch_kernel(embedding_kernel<bf16>, n_tokens, threads, 0, stream, ids, (const bf16*)table, out, hidden, vocab, scale, positions, freq, error_flag);
+        launch_kernel(embedding_kernel<bf16>, n_tokens, threads, 0, stream, ids, (const bf16*)table, out, hidden, vocab, scale, positions, freq, (const bf16*)pos_table, pos_rows, error_flag);
     else
         return KL_ERR_BAD_DTYPE;
     KL_LAUNCH_CHECK();
@@ -268,15 +284,18 @@ KL_API int kl_add_rmsnorm(float* residual, const void* delta, const float* parti
     return KL_OK;
 }
 
-KL_API int kl_swiglu(const void* gate_up, void* out, int tokens, int inter, int gelu, int dtype, cudaStream_t stream) {
+// kind, limit, alpha, shift: see swiglu_kernel.
+KL_API int kl_swiglu(const void* gate_up, void* out, int tokens, int inter, int kind, float limit, float alpha, float shift, int dtype,
+                     cudaStream_t stream) {
     if (tokens <= 0) return KL_OK;
+    if (kind < 1 || kind > 4) return KL_ERR_BAD_SIZE;
     const size_t n = (size_t)tokens * inter;
     const int threads = 256;
     const int blocks = kl::strided_grid(n, threads, 16);
     if (dtype == KL_F32)
-        launch_kernel(swiglu_kernel<float>, blocks, threads, 0, stream, (const float*)gate_up, (float*)out, tokens, inter, gelu);
+        launch_kernel(swiglu_kernel<float>, blocks, threads, 0, stream, (const float*)gate_up, (float*)out, tokens, inter, kind, limit, alpha, shift);
     else if (dtype == KL_BF16)
-        launch_kernel(swiglu_kernel<bf16>, blocks, threads, 0, stream, (const bf16*)gate_up, (bf16*)out, tokens, inter, gelu);
+        launch_kernel(swiglu_kernel<bf16>, blocks, threads, 0, stream, (const bf16*)gate_up, (bf16*)out, tokens, inter, kind, limit, alpha, shift);
     else
         return KL_ERR_BAD_DTYPE;
     KL_LAUNCH_CHECK();

@@ -121,3 +121,20 @@ KL_API int kl_short_conv(const void* x, long long ld_x, const float* w, const fl
     }
     return KL_OK;
 }
+
+// The state alone after a step (a caller whose own kernel convolved): the last taps - 1 rows of x, `channels` wide, per sequence.
+KL_API int kl_short_conv_state(const void* x, long long ld_x, int taps, float* state, long long ld_state, const int* cu_tokens,
+                               const int* seq_slots, int n_seqs, int channels, int dtype, cudaStream_t stream) {
+    if (n_seqs <= 0 || channels <= 0 || taps <= 1) return KL_OK;
+    if (taps > SC_MAX_TAPS || n_seqs > 65535) return KL_ERR_BAD_SIZE;
+    const int threads = channels >= 256 ? 256 : ((channels + 31) / 32) * 32;
+    const dim3 grid((channels + threads - 1) / threads, n_seqs);
+    if (dtype == KL_F32)
+        launch_kernel(short_conv_state_kernel<float>, grid, threads, 0, stream, (const float*)x, ld_x, taps, state, ld_state, cu_tokens, seq_slots, channels);
+    else if (dtype == KL_BF16)
+        launch_kernel(short_conv_state_kernel<bf16>, grid, threads, 0, stream, (const bf16*)x, ld_x, taps, state, ld_state, cu_tokens, seq_slots, channels);
+    else
+        return KL_ERR_BAD_DTYPE;
+    KL_LAUNCH_CHECK();
+    return KL_OK;
+}

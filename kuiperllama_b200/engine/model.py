@@ -28,6 +28,8 @@ def model_manifest(spec: ModelSpec) -> Dict[str, TensorDecl]:
             m.update(part_class(family, ps.kind).manifest(ps, layer.prefix))
         if layer.position is not None:
             m.update(part_class("position", layer.position.kind).manifest(layer.position, layer.prefix))
+    if spec.embedding_position is not None:
+        m.update(part_class("position", spec.embedding_position.kind).manifest(spec.embedding_position, ""))
     m.update(part_class("norm", spec.final_norm.kind).manifest(spec.final_norm, spec.final_norm_prefix))
     if spec.lm_head_name is not None:
         m[spec.lm_head_name] = TensorDecl((spec.vocab_size, spec.hidden_size))
@@ -48,6 +50,9 @@ class DecoderModel:
         dev, dt = runtime.device, runtime.dtype
         self.embedding = tensors[spec.embedding_name].to(device=dev, dtype=dt).contiguous()
         self.blocks = [self._build_layer(layer, tensors) for layer in spec.layers]
+        self.embedding_position = None
+        if spec.embedding_position is not None:
+            self.embedding_position = part_class("position", spec.embedding_position.kind)(spec.embedding_position, "", tensors, runtime)
         self.final_norm = part_class("norm", spec.final_norm.kind)(spec.final_norm, spec.final_norm_prefix, tensors, runtime)
         if spec.lm_head_name is None:
             self.lm_head = Linear(self.embedding, runtime)    # tied: the same storage, no copy
@@ -103,15 +108,16 @@ class DecoderModel:
 
     # ------------------------------------------------------------------ forward
     def hidden_states(self, step: StepContext, cache: SequenceCache) -> Tuple[torch.Tensor, Optional[torch.Tensor]]:
-        """Run embedding and all scheduled layers: the float32 residual stream and the last
+        """Run embedding and all scheduled layers: the float32 residual stream (or streams) and the last
         feed-forward's output that is still to be added to it."""
         step.allow_stream_fusion = self.stream_fusion and step.is_decode
         step.shared.clear()
         residual = torch.empty((step.n_tokens, self.spec.hidden_size), dtype=torch.float32, device=self.runtime.device)
-        position = getattr(self.blocks[self.spec.schedule[0].layer], "position", None)
+        position = self.embedding_position or getattr(self.blocks[self.spec.schedule[0].layer], "position", None)
         ops.embedding(step.token_ids[:step.n_tokens], self.embedding, residual, self.error_flag,
                       scale=1.0 if self.spec.embedding_multiplier is None else float(self.spec.embedding_multiplier),
-                      positions=step.positions, freq=position.embedding_frequencies() if position is not None else None)
+                      positions=step.positions, freq=position.embedding_frequencies() if position is not None else None,
+                      position_table=position.embedding_table() if position is not None else None)
         if position is not None:
             position.add_to_embeddings(residual, step)
         pending = None
@@ -148,6 +154,8 @@ class DecoderModel:
         yield self.embedding
         yield self.lm_head.weight
         parts = [p for b in self.blocks for p in vars(b).values() if isinstance(p, Part)]
+        if self.embedding_position is not None:
+            parts.append(self.embedding_position)
         for part in parts:                       # grows by the parts inside parts
             for v in vars(part).values():
                 if isinstance(v, Part) and v not in parts:

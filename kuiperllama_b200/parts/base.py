@@ -4,8 +4,8 @@ A part is built from a ``PartSpec`` (its sizes and constants), a tensor-name pre
 loaded tensors and the run's ``Runtime`` (device and compute dtype).  It never sees the
 model's configuration, so no part knows which model it is in.  A new part is a class with
 the interface below, registered under a name with ``register_mixer`` / ``register_feed_forward``
-/ ``register_norm`` / ``register_position`` / ``register_gate`` / ``register_arrangement``; a ``LayerSpec`` then
-names it.
+/ ``register_norm`` / ``register_position`` / ``register_gate`` / ``register_streams`` / ``register_arrangement``; a ``LayerSpec``
+then names it.
 
 ExiledOfCode/KuiperLLama's counterpart is its op layer (kuiper/include/op/layer.h:25-188):
 layers with stored inputs and outputs wired by the model class, with eps, theta and head
@@ -142,6 +142,17 @@ class DeltaSum:
     second: Optional[torch.Tensor] = None
 
 
+@dataclass
+class StreamsDelta:
+    """A sublayer's result on its way into several residual streams: x'_t = sum_s mix[s, t] x_s + out_weights[t] * value, all
+    streams at once from the old ones (``links``: the connection whose weights these are).  ``target``: float32
+    [n_tokens, S, hidden], where the new streams are kept; the old ones may be one row for all of them (a model's embeddings).
+    The norm that reads the streams next does it in its own kernel (``ops.stream_norm``)."""
+    value: torch.Tensor                       # [n_tokens, hidden] in the compute dtype, or float32 pieces [P, n_tokens, hidden]
+    links: "StreamLinks"
+    target: torch.Tensor
+
+
 class Part:
     """Base of all parts."""
 
@@ -179,12 +190,16 @@ class PositionEncoding(Part):
     returns the inverse frequencies and the rotated width) or changes the embeddings before
     the first layer (``add_to_embeddings``), or both.  One that adds a sinusoid to the embeddings gives its
     frequencies (``embedding_frequencies``, float32 [2, ceil(hidden / 2)]: every pair's frequency and what its rounding left
-    over), and the embedding kernel adds it itself."""
+    over), one that adds learned vectors gives their table (``embedding_table``, [positions, hidden] in the compute dtype), and the
+    embedding kernel adds them itself."""
 
     def rotary(self) -> Optional[tuple]:
         return None
 
     def embedding_frequencies(self) -> Optional[torch.Tensor]:
+        return None
+
+    def embedding_table(self) -> Optional[torch.Tensor]:
         return None
 
     def add_to_embeddings(self, residual: torch.Tensor, step: StepContext) -> None:
@@ -233,6 +248,17 @@ class ResidualGate(Part):
         raise NotImplementedError
 
 
+class StreamLinks(Part):
+    """How one sublayer reads several residual streams and writes into them: ``streams`` of them, ``in_weights`` float32
+    [S] (the sublayer's input is their sum by these), ``mix`` float32 [S, S] ([from, to]) and ``out_weights`` float32 [S] (see
+    ``StreamsDelta``)."""
+
+    streams: int
+    in_weights: torch.Tensor
+    mix: torch.Tensor
+    out_weights: torch.Tensor
+
+
 class FeedForward(Part):
     """``forward(x, step)``: [n_tokens, hidden] -> [n_tokens, hidden], token by token (or
     float32 partial sums [S, n_tokens, hidden], as a mixer may)."""
@@ -247,7 +273,7 @@ class FeedForward(Part):
 # ----------------------------------------------------------------------------- registries
 
 _REGISTRIES: Dict[str, Dict[str, type]] = {"mixer": {}, "feed_forward": {}, "norm": {}, "position": {},
-                                           "arrangement": {}, "gate": {}}
+                                           "arrangement": {}, "gate": {}, "streams": {}}
 
 
 def _register(family: str, name: str) -> Callable[[type], type]:
@@ -263,6 +289,7 @@ def register_norm(name: str): return _register("norm", name)
 def register_position(name: str): return _register("position", name)
 def register_arrangement(name: str): return _register("arrangement", name)
 def register_gate(name: str): return _register("gate", name)
+def register_streams(name: str): return _register("streams", name)
 
 
 def part_class(family: str, name: str) -> type:

@@ -6,7 +6,7 @@ from typing import Optional, Tuple
 import torch
 
 from ..cache import CacheView
-from .base import DeltaSum, FeedForward, Mixer, Norm, NormedLazy, PostNormed, ResidualGate, StepContext, StreamSink, register_arrangement
+from .base import DeltaSum, FeedForward, Mixer, Norm, NormedLazy, PostNormed, ResidualGate, StepContext, StreamLinks, StreamSink, StreamsDelta, register_arrangement
 
 
 @register_arrangement("pre_norm")
@@ -131,3 +131,42 @@ class ParallelBlock:
         if self.feed_forward is None:
             return residual, mixed
         return residual, DeltaSum(mixed, self.feed_forward.forward(h2, step))
+
+
+@register_arrangement("streams")
+class StreamsBlock:
+    """The pre-norm block between several residual streams:
+
+        u = sum_s a[s] x_s;  x_t <- sum_s M[s, t] x_s + b[t] mixer(norm1(u));  then the same with the feed-forward and its
+        own a, M, b (left out without a feed-forward)
+
+    with a, M and b from each sublayer's ``StreamLinks``.  The streams are float32 [n, S, hidden]; the first block of a model
+    receives one row per token, which all of its streams are.  As in the pre-norm block no update runs as a kernel of its own: a
+    sublayer's result travels as ``StreamsDelta`` to the norm that reads the streams next, whose kernel mixes and writes the
+    streams, combines them and norms the combination.  KuiperLLama has one stream (kuiper/source/model/llama3.cpp:155-164)."""
+
+    def __init__(self, mixer_norm: Norm, mixer: Mixer, feed_forward_norm: Optional[Norm], feed_forward: Optional[FeedForward],
+                 mixer_streams: StreamLinks = None, feed_forward_streams: Optional[StreamLinks] = None):
+        self.mixer_norm, self.mixer = mixer_norm, mixer
+        self.feed_forward_norm, self.feed_forward = feed_forward_norm, feed_forward
+        self.mixer_streams, self.feed_forward_streams = mixer_streams, feed_forward_streams
+        if mixer_streams is None or (feed_forward is not None and feed_forward_streams is None):
+            raise ValueError("a block between several streams needs the links of each of its sublayers")
+        if not hasattr(mixer_norm, "forward_streams") or (feed_forward is not None and not hasattr(feed_forward_norm, "forward_streams")):
+            raise ValueError("a block between several streams needs norms that read them (rmsnorm)")
+
+    @staticmethod
+    def _result(y, links: StreamLinks, streams: torch.Tensor) -> StreamsDelta:
+        target = streams
+        if streams.dim() == 2:                               # one row for all of them until now
+            target = torch.empty((streams.shape[0], links.streams, streams.shape[1]), dtype=streams.dtype, device=streams.device)
+        return StreamsDelta(y, links, target)
+
+    def forward(self, residual: torch.Tensor, pending, step: StepContext, cache: CacheView):
+        step.residual_sink = None
+        h, residual = self.mixer_norm.forward_streams(residual, pending, self.mixer_streams)
+        pending = self._result(self.mixer.forward(h, step, cache), self.mixer_streams, residual)
+        if self.feed_forward is None:
+            return residual, pending
+        h, residual = self.feed_forward_norm.forward_streams(residual, pending, self.feed_forward_streams)
+        return residual, self._result(self.feed_forward.forward(h, step), self.feed_forward_streams, residual)

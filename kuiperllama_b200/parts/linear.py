@@ -94,16 +94,20 @@ class StackedInput:
             self._pieces.append((None, torch.zeros((gap, like.shape[1]), dtype=like.dtype, device=like.device)))
             self.total += gap
 
+    def close(self) -> None:
+        """No further projection may be added: ``total`` is the product's final width."""
+        if self.linear is None:
+            self._pad()
+            self.linear = Linear(torch.cat([w for _, w in self._pieces], dim=0), self.runtime)
+            self._pieces = []
+
     def column(self, name: str) -> int:
         return self.columns[name][0]
 
     def forward(self, x: torch.Tensor, allow_partials: bool = False) -> torch.Tensor:
         """[m, total].  With ``allow_partials`` the result may be float32 pieces [S, m, total] (see ``Linear.forward``), which the
         caller's kernel adds; ``view`` is then not to be used."""
-        if self.linear is None:
-            self._pad()
-            self.linear = Linear(torch.cat([w for _, w in self._pieces], dim=0), self.runtime)
-            self._pieces = []
+        self.close()
         self.rows = x
         self.last = self.linear.forward(x, allow_partials=allow_partials)
         return self.last

@@ -23,11 +23,16 @@ class MoEFeedForward(FeedForward):
                    f_e = W_down[e] (g * sigmoid(alpha * g) * (u + shift))          (no clamp when limit is None)
         out = sum over the chosen e of s_e * f_e     (the weights are divided by their sum + ``renorm_eps`` if ``renormalise``)
 
+    ``identity`` = I: the router scores I more experts, which come last; an identity expert's result is the input row n itself, it
+    has no tensors and joins no product.
+
     With ``gated`` False an expert has no gate: f_e = W_down[e] act(W_up[e] n) with ``activation`` one of the element-wise
     activations (``ops.ACTIVATIONS``).  ``names['router_bias']``: a bias per expert joins the router's logits (32 bits).  With
     ``renormalise`` and no ``renorm_eps`` the weights are the softmax over the chosen logits alone.  ``shared_size``: one more
     expert of that size and of the same form (``names['shared_up']``, ``names['shared_down']``, gated also
-    ``names['shared_gate']``) runs for every token and is added, as a second float32 piece.  ``scores`` "sigmoid": s = sigmoid(z),
+    ``names['shared_gate']``, with ``shared_limit`` for its clamp) runs for every token and is added; ``names['shared_scale']``
+    [1, hidden]: it is first multiplied by sigmoid of that row's product with n, one number per token (the row rides on the
+    router's product).  ``scores`` "sigmoid": s = sigmoid(z),
     each expert by itself; ``names['correction']``: a number per expert that joins the scores for the choice (of groups
     too) but not for the weights; ``router_scale`` multiplies the weights.
 
@@ -37,14 +42,15 @@ class MoEFeedForward(FeedForward):
     Routing stays on the device (``ops.moe_route`` / ``moe_plan``): the (token, choice) pairs are sorted by
     expert into a list padded to whole tiles, one grouped product makes gate, up and the activation for
     the whole list, one more the down projection, and ``moe_combine`` adds each token's results in the
-    order of its choices in 32 bits.  The result is handed on as one float32 piece.  The grouped products run on the
+    order of its choices, identity experts and a gated shared expert in 32 bits.  The result is handed on as one float32 piece (an
+    ungated shared expert is a second one).  The grouped products run on the
     tensor cores where the sizes allow (bfloat16, expert size % 64, hidden size % 8): tokens as tile rows from
     ``TENSOR_CORE_ROWS_PER_EXPERT`` rows per expert on, weights as tile rows below (a decode step); on FMA kernels
     otherwise (float32, odd sizes).
 
     Spec: ``hidden_size``, ``experts``, ``top``, ``expert_size``, ``limit``, ``alpha``, ``shift``, ``renormalise``,
     ``renorm_eps``, ``groups``, ``keep_groups``, ``group_top``, ``scores``, ``router_scale``, ``gated``, ``activation``,
-    ``shared_size``, ``names``: router and, with ``{e}`` for the
+    ``shared_size``, ``shared_limit``, ``identity``, ``names``: router and, with ``{e}`` for the
     expert's number, gate, up, down.  KuiperLLama's only feed-forward is
     the dense SwiGLU (kuiper/source/model/llama3.cpp:692-718)."""
 
@@ -57,11 +63,12 @@ class MoEFeedForward(FeedForward):
     @classmethod
     def manifest(cls, spec: PartSpec, prefix: str) -> Dict[str, TensorDecl]:
         hid, E, ff, n = spec["hidden_size"], spec["experts"], spec["expert_size"], spec["names"]
-        m = {prefix + n["router"]: TensorDecl((E, hid))}
+        scored = E + int(spec.get("identity") or 0)
+        m = {prefix + n["router"]: TensorDecl((scored, hid))}
         if n.get("router_bias"):
-            m[prefix + n["router_bias"]] = TensorDecl((E,), role="vector")
+            m[prefix + n["router_bias"]] = TensorDecl((scored,), role="vector")
         if n.get("correction"):
-            m[prefix + n["correction"]] = TensorDecl((E,), role="vector")
+            m[prefix + n["correction"]] = TensorDecl((scored,), role="vector")
         for e in range(E):
             if spec.get("gated", True):
                 m[prefix + n["gate"].format(e=e)] = TensorDecl((ff, hid))
@@ -72,24 +79,32 @@ class MoEFeedForward(FeedForward):
                 m[prefix + n["shared_gate"]] = TensorDecl((spec["shared_size"], hid))
             m[prefix + n["shared_up"]] = TensorDecl((spec["shared_size"], hid))
             m[prefix + n["shared_down"]] = TensorDecl((hid, spec["shared_size"]))
+            if n.get("shared_scale"):
+                m[prefix + n["shared_scale"]] = TensorDecl((1, hid))
         return m
 
     def __init__(self, spec, prefix, tensors, runtime: Runtime):
         super().__init__(spec, prefix, tensors, runtime)
         self.hidden, self.E, self.top, self.ff = (int(spec[k]) for k in ("hidden_size", "experts", "top", "expert_size"))
-        if not 0 < self.top <= self.E <= ops.MOE_MAX_EXPERTS:
-            raise ValueError(f"{self.top} of {self.E} experts: the routing kernels take up to {ops.MOE_MAX_EXPERTS} experts")
+        self.identity = int(spec.get("identity") or 0)
+        self.scored = self.E + self.identity                     # what the router scores: identity experts come last
+        if not 0 < self.top <= self.scored <= ops.MOE_MAX_EXPERTS:
+            raise ValueError(f"{self.top} of {self.scored} experts: the routing kernels take up to {ops.MOE_MAX_EXPERTS} experts")
         limit = spec.get("limit")
         self.activation = (float(limit) if limit is not None else 0.0, float(spec.get("alpha", 1.0)), float(spec.get("shift", 0.0)))
         self.renormalise = bool(spec.get("renormalise", False))
         self.renorm_eps = float(spec.get("renorm_eps", 0.0))
         self.groups, self.keep_groups = int(spec.get("groups", 1)), int(spec.get("keep_groups", 1))
-        if self.E % self.groups or not 1 <= self.keep_groups <= self.groups or self.top > self.keep_groups * (self.E // self.groups):
-            raise ValueError(f"{self.E} experts in {self.groups} groups of which {self.keep_groups} are kept do not hold {self.top} choices")
+        if self.scored % self.groups or not 1 <= self.keep_groups <= self.groups or self.top > self.keep_groups * (self.scored // self.groups):
+            raise ValueError(f"{self.scored} experts in {self.groups} groups of which {self.keep_groups} are kept do not hold {self.top} choices")
         n = spec["names"]
         dev, dt = runtime.device, runtime.dtype
         get = lambda key, e: tensors[prefix + n[key].format(e=e)].to(device=dev, dtype=dt)
-        self.router = Linear(tensors[prefix + n["router"]], runtime)
+        router = tensors[prefix + n["router"]]
+        self.shared_scale = bool(spec.get("shared_size")) and bool(n.get("shared_scale"))
+        if self.shared_scale:
+            router = torch.cat([router.to(device=dev, dtype=dt), tensors[prefix + n["shared_scale"]].to(device=dev, dtype=dt)])
+        self.router = Linear(router, runtime)
         self.router_bias = None
         if n.get("router_bias"):
             self.router_bias = tensors[prefix + n["router_bias"]].to(device=dev, dtype=torch.float32).contiguous()
@@ -121,12 +136,16 @@ class MoEFeedForward(FeedForward):
         self.shared_size = int(spec.get("shared_size") or 0)
         self.shared = None
         if self.shared_size and self.gated:
-            if self.activation != (0.0, 1.0, 0.0):
-                raise ValueError("a shared expert beside gated experts has their plain silu form")
             names = {"gate": n["shared_gate"], "up": n["shared_up"], "down": n["shared_down"]}
-            self.shared = SwiGLUFeedForward(PartSpec("swiglu", {"hidden_size": self.hidden, "intermediate_size": self.shared_size, "names": names}),
+            form = {"activation": "silu"}
+            shared_limit = spec.get("shared_limit", limit)
+            if self.activation[1:] != (1.0, 0.0) or shared_limit is not None:
+                form = {"activation": "clamped", "limit": shared_limit, "alpha": self.activation[1], "shift": self.activation[2]}
+            self.shared = SwiGLUFeedForward(PartSpec("swiglu", dict(form, hidden_size=self.hidden, intermediate_size=self.shared_size, names=names)),
                                             prefix, tensors, runtime)
         elif self.shared_size:
+            if self.shared_scale:
+                raise ValueError("a shared expert's factor goes with gated experts")
             self.shared_up = Linear(tensors[prefix + n["shared_up"]], runtime)
             self.shared_down = Linear(tensors[prefix + n["shared_down"]], runtime)
 
@@ -138,7 +157,8 @@ class MoEFeedForward(FeedForward):
         if isinstance(x, NormedLazy):
             x = x.dense()
         n, dev, dt = step.n_tokens, x.device, self.runtime.dtype
-        logits = self.router.forward(x, out_dtype=torch.float32)
+        scored = self.router.forward(x, out_dtype=torch.float32)
+        logits = scored[:, :self.scored]
         choice, weight = ops.moe_route(logits, self.top, self.renormalise, self.groups, self.keep_groups, self.renorm_eps,
                                        bias=self.router_bias, scores=self.scores, correction=self.correction,
                                             group_top=self.group_top, scale=self.router_scale)
@@ -175,11 +195,11 @@ class MoEFeedForward(FeedForward):
                                  interleaved=self.tensor_cores and self.gated, activation=self.fused_act)
                 self._activate(act)
                 ops.grouped_gemm(act, self.down, res, a_rows=None, tile_group=tile_group, tile_rows=tile)
-        out = torch.empty((2 if self.shared_size else 1, n, self.hidden), dtype=torch.float32, device=dev)
-        ops.moe_combine(res, pair_pos, weight, out[0])
-        if self.shared is not None:
-            self.shared.forward_into(x, out[1][:x.shape[0]])
-        elif self.shared_size:
+        own_piece = self.shared_size > 0 and self.shared is None
+        out = torch.empty((2 if own_piece else 1, n, self.hidden), dtype=torch.float32, device=dev)
+        ops.moe_combine(res, pair_pos, weight, out[0], x=x if self.identity else None, shared=None if self.shared is None else self.shared.result(x),
+                        shared_gate=scored[:, self.scored] if self.shared_scale else None)
+        if own_piece:
             # the expert every token takes: its down product writes the second float32 piece
             up = self.shared_up.forward(x)
             ops.activation(up, up, self.act_kind)

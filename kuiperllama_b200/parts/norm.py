@@ -8,7 +8,7 @@ import torch
 from ..config.spec import PartSpec
 from ..csrc import ops
 from ..weights.loader import TensorDecl
-from .base import Accumulated, DeltaSum, Norm, NormedLazy, PostNormed, Runtime, register_norm
+from .base import Accumulated, DeltaSum, Norm, NormedLazy, PostNormed, Runtime, StreamLinks, StreamsDelta, register_norm
 
 
 @register_norm("rmsnorm")
@@ -41,6 +41,12 @@ class RMSNorm(Norm):
             return chain_forward(self, residual, delta, rows)
         if isinstance(delta, DeltaSum):
             return self.forward_pair(residual, delta, None, rows)[0]
+        if isinstance(delta, StreamsDelta):                  # a norm of the streams' sum; the streams are not needed after it
+            n_out = rows.numel() if rows is not None else residual.shape[0]
+            out = torch.empty((n_out, self.size), dtype=self.runtime.dtype, device=residual.device)
+            ops.stream_norm(residual, delta.value, out, self.weight, self.eps, mix=delta.links.mix, out_weights=delta.links.out_weights,
+                            n_streams=delta.links.streams, rows=rows)
+            return out
         if isinstance(delta, Accumulated):
             # the stream holds the sum already; if the rows times this norm's weight came with it,
             # the product that follows only has to apply 1 / rms
@@ -51,6 +57,18 @@ class RMSNorm(Norm):
         out = torch.empty((n_out, self.size), dtype=self.runtime.dtype, device=residual.device)
         ops.add_rmsnorm(residual, delta, self.weight, out, self.eps, rows)
         return out
+
+
+def _forward_streams(self, residual: torch.Tensor, delta: Optional[StreamsDelta], links: StreamLinks):
+    """(this norm of the sublayer input that ``links`` makes of the streams once ``delta`` is in them, the streams).  ``residual``:
+    [n, S, hidden], or [n, hidden] where every stream is still that row."""
+    out = torch.empty((residual.shape[0], self.size), dtype=self.runtime.dtype, device=residual.device)
+    if delta is None:
+        ops.stream_norm(residual, None, out, self.weight, self.eps, in_weights=links.in_weights, n_streams=links.streams)
+        return out, residual
+    ops.stream_norm(residual, delta.value, out, self.weight, self.eps, mix=delta.links.mix, out_weights=delta.links.out_weights,
+                    in_weights=links.in_weights, write=delta.target, n_streams=links.streams)
+    return out, delta.target
 
 
 def _forward_pair(self, residual: torch.Tensor, delta, other: Optional["RMSNorm"], rows: Optional[torch.Tensor] = None):
@@ -66,6 +84,7 @@ def _forward_pair(self, residual: torch.Tensor, delta, other: Optional["RMSNorm"
 
 
 RMSNorm.forward_pair = _forward_pair
+RMSNorm.forward_streams = _forward_streams
 
 
 def chain_forward(norm: Norm, residual: torch.Tensor, delta, rows: Optional[torch.Tensor]) -> torch.Tensor:
@@ -89,6 +108,10 @@ def add_to_stream(residual: torch.Tensor, delta) -> None:
     """Add a pending delta to the stream without a norm after it (what a caller that wants the
     stream itself does after the last block)."""
     if delta is None:
+        return
+    if isinstance(delta, StreamsDelta):                      # the new streams are in ``delta.target``
+        ops.stream_norm(residual, delta.value, None, None, 0.0, mix=delta.links.mix, out_weights=delta.links.out_weights, write=delta.target,
+                        n_streams=delta.links.streams)
         return
     if isinstance(delta, DeltaSum):
         ops.pair_rmsnorm(residual, (delta.first, delta.second), None, None, None, None, 0.0,

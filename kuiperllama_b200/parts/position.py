@@ -1,11 +1,13 @@
-"""Position encodings: the tables of inverse frequencies of a rotation, and a sinusoid added to the embeddings."""
+"""Position encodings: the tables of inverse frequencies of a rotation, and a sinusoid or learned vectors added to the embeddings."""
 from __future__ import annotations
 
 import math
-from typing import List, Optional
+from typing import Dict, List, Optional
 
 import torch
 
+from ..config.spec import PartSpec
+from ..weights.loader import TensorDecl
 from .base import PositionEncoding, Runtime, register_position
 
 
@@ -111,3 +113,21 @@ class SinusoidalPosition(PositionEncoding):
 
     def embedding_frequencies(self):
         return self.frequencies
+
+
+@register_position("learned")
+class LearnedPosition(PositionEncoding):
+    """A learned vector per position, added to the embeddings before the first layer (unscaled).  The embedding kernel adds it.
+    Spec: ``hidden_size``, ``positions`` (rows of the table) and the tensor's ``name``.  KuiperLLama knows rotations
+    alone (rope_kernel.cu:5-49)."""
+
+    @classmethod
+    def manifest(cls, spec: PartSpec, prefix: str) -> Dict[str, TensorDecl]:
+        return {prefix + spec["name"]: TensorDecl((spec["positions"], spec["hidden_size"]))}
+
+    def __init__(self, spec, prefix, tensors, runtime: Runtime):
+        super().__init__(spec, prefix, tensors, runtime)
+        self.table = tensors[prefix + spec["name"]].to(device=runtime.device, dtype=runtime.dtype).contiguous()
+
+    def embedding_table(self):
+        return self.table

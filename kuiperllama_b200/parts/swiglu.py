@@ -18,8 +18,9 @@ class SwiGLUFeedForward(FeedForward):
     (ExiledOfCode/KuiperLLama kuiper/source/model/llama3.cpp:692-718, swiglu_kernel.cu:18-21;
     gate = w1, up = w3, down = w2, tools/export_llama3.py:583-585).  Gate and up are stacked
     into one matrix at load (and the activation is applied in that product's epilogue where the
-    tensor-core kernel runs).  ``activation`` "gelu_tanh" puts the tanh form of gelu in silu's place.  Spec: ``hidden_size``,
-    ``intermediate_size``, ``activation`` ("silu"), ``names``."""
+    tensor-core kernel runs).  ``activation`` "gelu_tanh" puts the tanh form of gelu in silu's place, "relu" a relu; "clamped" is
+    min(g, limit) * sigmoid(alpha * min(g, limit)) * (clamp(u, -limit, limit) + shift) (no clamp when ``limit`` is None).  Spec:
+    ``hidden_size``, ``intermediate_size``, ``activation`` ("silu"), for "clamped" ``limit``, ``alpha`` (1), ``shift`` (0), ``names``."""
 
     accepts_lazy_norm = True
     may_accumulate = True
@@ -34,8 +35,11 @@ class SwiGLUFeedForward(FeedForward):
         super().__init__(spec, prefix, tensors, runtime)
         self.hidden, self.inter = int(spec["hidden_size"]), int(spec["intermediate_size"])
         self.activation = str(spec.get("activation") or "silu")
-        if self.activation not in ops.GATED_ACTIVATIONS:
-            raise ValueError(f"unknown activation {self.activation!r} (known: {', '.join(sorted(ops.GATED_ACTIVATIONS))})")
+        if self.activation == "clamped":
+            limit = spec.get("limit")
+            self.activation = (0.0 if limit is None else float(limit), float(spec.get("alpha", 1.0)), float(spec.get("shift", 0.0)))
+        elif self.activation not in ops.GATED_ACTIVATIONS:
+            raise ValueError(f"unknown activation {self.activation!r} (known: {', '.join(sorted(ops.GATED_ACTIVATIONS))}, clamped)")
         n = spec["names"]
         dev, dt = runtime.device, runtime.dtype
         gate, up = (tensors[prefix + n[k]].to(device=dev, dtype=dt) for k in ("gate", "up"))
@@ -55,9 +59,9 @@ class SwiGLUFeedForward(FeedForward):
             x = x.dense()
         return self.down.forward(self._activated(x), allow_partials=True, sink=getattr(step, "residual_sink", None))
 
-    def forward_into(self, x: torch.Tensor, out: torch.Tensor) -> None:
-        """The same into ``out`` (a tensor of the caller's, float32 or the compute dtype)."""
-        self.down.forward(self._activated(x), out=out)
+    def result(self, x: torch.Tensor) -> torch.Tensor:
+        """The same for a caller that adds it itself: rows in the compute dtype, or float32 pieces."""
+        return self.down.forward(self._activated(x), allow_partials=True)
 
     def _activated(self, x: torch.Tensor) -> torch.Tensor:
         act = torch.empty((x.shape[0], self.inter), dtype=self.runtime.dtype, device=x.device)

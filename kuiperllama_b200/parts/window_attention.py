@@ -1,7 +1,7 @@
 """Grouped-query attention over a window of recent keys, with the options that softmax attention in the plain
 Llama form does not have: biased projections, a norm on q and k heads or over the whole projection, interleaved
 rotary pairs, values of another size, a sink, sigmoid weights, pooled blocks before the window, chunks, a bias by
-distance, and values mixed with another layer's."""
+distance, short convolutions behind the projections, and values mixed with another layer's."""
 from __future__ import annotations
 
 import math
@@ -9,7 +9,7 @@ from typing import Dict, Optional
 
 import torch
 
-from ..cache import CacheView, KVRequest
+from ..cache import CacheView, KVRequest, StateRequest
 from ..config.spec import PartSpec
 from ..csrc import ops
 from ..weights.loader import TensorDecl
@@ -52,18 +52,24 @@ class WindowAttentionMixer(Mixer):
     table[bucket(i - j), h] after the scaling (``distance_buckets``).  ``value_mix``: "keep" leaves the layer's values as
     projected for later layers of the step; "mix" caches (1 - lambda) v + lambda v_kept, lambda = ``names['value_mix']``, one number.
 
+    ``conv`` = taps: every channel of q, k and v passes a causal filter of so many taps over time directly behind its projection
+    (``names['q_conv']``, ``['k_conv']``, ``['v_conv']`` [channels, taps]; y_t = sum_j w[:, j] u_(t - taps + 1 + j), nothing before the
+    sequence's start), before rotation and value mixing; the last taps - 1 projected rows are state of the sequence.  ``sink_score``: a
+    number s, the same for every head and not learned: exp(s) joins the softmax's denominator.
+
     One product makes q | k | v; ``ops.qk_prepare`` does bias, rotation, norm and the cache write in one kernel;
-    ``ops.qk_row_prepare`` does norm over rows, value mixing and cache write; ``ops.pool_blocks`` writes the means of the blocks
+    ``ops.qk_row_prepare`` does norm over rows, value mixing and cache write; ``ops.qkv_conv`` does convolutions, rotation, value mixing
+    and cache write; ``ops.pool_blocks`` writes the means of the blocks
     that the step completes.  Chunks, a distance bias and values of another size run on the tensor cores for bfloat16 key and
-    value sizes of 32, 64 and 128 (``ops.attention_chunked_mma``).  Softmax without pooled blocks
+    value sizes of 32, 64, 96 and 128 (``ops.attention_chunked_mma``), with a sink too.  Softmax without pooled blocks
     runs on the attention kernels of ``AttentionMixer`` where they take the sizes; a sink, sigmoid weights and pooled blocks
     are options of the windowed tensor-core kernel (bfloat16, equal key and value sizes of 64 or 128, groups of up to 16
     heads); everything else runs on the plain kernels.
 
     Spec: ``hidden_size``, ``num_heads``, ``num_kv_heads``, ``head_dim``, ``value_dim``, ``scale``, ``window``, ``values``
     ("own" | "keys"), ``weights`` ("softmax" | "sigmoid"), ``pool`` (None), ``head_norm`` (None | {"eps"}), ``row_norm``
-    (None | {"eps"}), ``chunk``, ``distance_bias``, ``value_mix`` (None | "keep" | "mix"), ``names`` (q, k, o and optionally v,
-    q_bias, k_bias, v_bias, q_norm, k_norm, sink, head_bias, distance_bias, value_mix).  KuiperLLama's attention is
+    (None | {"eps"}), ``chunk``, ``distance_bias``, ``value_mix`` (None | "keep" | "mix"), ``conv``, ``sink_score``, ``names`` (q, k, o and
+    optionally v, q_bias, k_bias, v_bias, q_norm, k_norm, sink, head_bias, distance_bias, value_mix, q_conv, k_conv, v_conv).  KuiperLLama's attention is
     the unbiased causal softmax over every earlier key (kuiper/source/model/llama3.cpp:610-639, mha_kernel.cu:61,74-106)."""
 
     KERNEL = "mma"                # "simt": the plain kernels also for bfloat16 (for comparisons)
@@ -89,6 +95,9 @@ class WindowAttentionMixer(Mixer):
             m[prefix + n["distance_bias"]] = TensorDecl((spec["distance_bias"]["rows"], H), role="vector")
         if spec.get("value_mix") == "mix":
             m[prefix + n["value_mix"]] = TensorDecl((), role="vector")
+        if spec.get("conv"):
+            for key, size in (("q_conv", H * hd), ("k_conv", KV * hd), ("v_conv", KV * vd)):
+                m[prefix + n[key]] = TensorDecl((size, spec["conv"]), role="vector")
         return m
 
     def __init__(self, spec, prefix, tensors, runtime: Runtime, position: Optional[PositionEncoding] = None):
@@ -114,7 +123,13 @@ class WindowAttentionMixer(Mixer):
         if self.value_mix not in (None, "keep", "mix"):
             raise ValueError(f"unknown value mixing {self.value_mix!r} (keep, mix)")
         row_norm = spec.get("row_norm")
-        self.by_rows = row_norm is not None or self.value_mix is not None      # prepared a whole projection at a time
+        self.taps = int(spec.get("conv") or 0)
+        if self.taps > ops.QKV_CONV_MAX_TAPS:
+            raise ValueError(f"the convolution kernel takes up to {ops.QKV_CONV_MAX_TAPS} taps, got {self.taps}")
+        rot = position.rotary() if position is not None else None
+        # convolutions, and mixed values beside a rotation, are prepared by the kernel that does all three
+        self.by_conv = self.taps > 0 or (self.value_mix is not None and rot is not None and row_norm is None)
+        self.by_rows = not self.by_conv and (row_norm is not None or self.value_mix is not None)      # prepared a whole projection at a time
         norm = spec.get("head_norm") if not self.by_rows else row_norm
         self.head_norm, self.eps = norm is not None, float(norm["eps"]) if norm is not None else 0.0
         n = spec["names"]
@@ -131,8 +146,17 @@ class WindowAttentionMixer(Mixer):
             reach = [int(math.ceil(max(largest, rows // 2))) + 1] + [int(c) for c in (self.chunk, self.window) if c]
             table = f32("distance_bias")
             self.distance_bias = table[distance_buckets(min(reach), rows, largest).to(dev)].T.contiguous()
-        if (self.chunk or self.distance_bias is not None) and (self.weights != "softmax" or self.pool or self.sink is not None):
-            raise ValueError("chunks and a distance bias go with a plain softmax: no sink, no sigmoid weights, no pooled blocks")
+        if spec.get("sink_score") is not None:
+            if self.sink is not None:
+                raise ValueError("a learned sink and a fixed one exclude each other")
+            self.sink = torch.full((self.H,), float(spec["sink_score"]), dtype=torch.float32, device=dev)
+        # sizes and options for which the kernels with values of their own size are asked
+        self.own_values = self.by_rows or self.by_conv or bool(self.chunk) or self.distance_bias is not None
+        if self.own_values and (self.weights != "softmax" or self.pool):
+            raise ValueError("chunks, a distance bias, convolutions and mixed values go with a softmax: no sigmoid weights, no pooled blocks")
+        if self.by_conv and (self.values_are_keys or row_norm is not None or spec.get("head_norm") is not None
+                             or any(t is not None for t in (self.q_bias, self.k_bias, self.v_bias))):
+            raise ValueError("convolutions come without biases, norms on q and k, and values that are keys")
         if self.by_rows and (self.values_are_keys or spec.get("head_norm") is not None or position is not None and position.rotary() is not None
                              or any(t is not None for t in (self.q_bias, self.k_bias, self.v_bias))):
             raise ValueError("a norm over the whole projection and mixed values come without biases, head norm, rotation and values that are keys")
@@ -144,11 +168,18 @@ class WindowAttentionMixer(Mixer):
         if not self.values_are_keys:
             self.inputs.add("v", tensors[prefix + n["v"]])
         self.o = Linear(tensors[prefix + n["o"]], runtime)
-        rot = position.rotary() if position is not None else None
         self.inv_freq, self.rotary_dim = rot if rot is not None else (None, 0)
-        if rot is not None and getattr(position, "magnitude", 1.0) != 1.0:
-            raise ValueError("this mixer's kernel rotates with unit magnitude")
+        self.magnitude = float(getattr(position, "magnitude", 1.0)) if rot is not None else 1.0
+        if self.magnitude != 1.0 and not self.by_conv:
+            raise ValueError("without convolutions this mixer's kernel rotates with unit magnitude")
         self.interleaved = getattr(position, "pairing", "half") == "interleaved"
+        self.conv_weight = None
+        if self.taps:
+            self.inputs.close()                             # the filters lie by column of the product
+            self.conv_weight = torch.zeros((self.taps, self.inputs.total), dtype=torch.float32, device=dev)
+            for key in ("q", "k", "v"):
+                c, w = self.inputs.columns[key]
+                self.conv_weight[:, c:c + w] = f32(key + "_conv").T
 
     def kv_request(self) -> Optional[KVRequest]:
         value_dim = None if self.vd == self.hd else self.vd
@@ -156,11 +187,14 @@ class WindowAttentionMixer(Mixer):
             return KVRequest(kv_heads=self.KV, head_dim=self.hd, kind="pooled", window=self.window, value_dim=value_dim, pool=self.pool)
         return KVRequest(kv_heads=self.KV, head_dim=self.hd, kind="full", window=self.window, value_dim=value_dim, chunk=self.chunk or None)
 
+    def state_request(self) -> Optional[StateRequest]:
+        return StateRequest(((self.taps - 1) * self.inputs.total,), torch.float32) if self.taps > 1 else None
+
     def forward(self, x, step: StepContext, cache: CacheView) -> torch.Tensor:
         if hasattr(x, "dense"):
             x = x.dense()
-        if self.by_rows or self.chunk or self.distance_bias is not None:
-            return self._forward_chunked(x, step, cache)
+        if self.own_values:
+            return self._forward_own_values(x, step, cache)
         n, dt = step.n_tokens, self.runtime.dtype
         proj = self.inputs.forward(x)
         q_col = self.inputs.column("q")
@@ -203,6 +237,16 @@ class WindowAttentionMixer(Mixer):
         n, dt = step.n_tokens, self.runtime.dtype
         write = cache.writable
         k_cache, v_cache = (cache.k, cache.v) if write else (None, None)
+        if self.by_conv:
+            if self.taps > 1 and not write:
+                raise ValueError("an execution with convolutions keeps a state of its own; it cannot read another one's cache")
+            proj = self.inputs.forward(x, allow_partials=step.is_decode)      # single tokens: the product's pieces, which the kernel adds
+            q, keep, first = self._mixed_values(x, step)
+            ops.qkv_conv(proj, self.inputs.column("q"), self.inputs.column("k"), self.inputs.column("v"), q, step, cache.block_table,
+                         k_cache, v_cache, self.H, self.KV, self.hd, self.vd, conv_weight=self.conv_weight, state=cache.state if self.taps > 1 else None,
+                         inv_freq=self.inv_freq, rotary_dim=self.rotary_dim, magnitude=self.magnitude, interleaved=self.interleaved,
+                         v_first=first, v_lambda=self.value_lambda, v_keep=keep)
+            return q
         if not self.by_rows:
             proj = self.inputs.forward(x)
             q_col = self.inputs.column("q")
@@ -213,19 +257,24 @@ class WindowAttentionMixer(Mixer):
                            k_norm_weight=self.k_norm)
             return proj[:, q_col:q_col + self.H * self.hd]
         proj = self.inputs.forward(x, allow_partials=True)          # few tokens: the product's pieces, which the kernel adds
-        make = torch.zeros if step.padded else torch.empty
-        q = make((n, self.H * self.hd), dtype=dt, device=x.device)
-        keep = first = None
-        if self.value_mix == "keep":
-            keep = step.shared["values"] = make((n, self.KV * self.vd), dtype=dt, device=x.device)
-        elif self.value_mix == "mix":
-            first = step.shared["values"]
+        q, keep, first = self._mixed_values(x, step)
         ops.qk_row_prepare(proj, self.inputs.column("q"), self.inputs.column("k"), self.inputs.column("v"), q, step, cache.block_table,
                            k_cache, v_cache, self.H, self.KV, self.hd, self.vd, norm=self.head_norm, eps=self.eps, q_norm_weight=self.q_norm,
                            k_norm_weight=self.k_norm, v_first=first, v_lambda=self.value_lambda, v_keep=keep)
         return q
 
-    def _forward_chunked(self, x, step: StepContext, cache: CacheView) -> torch.Tensor:
+    def _mixed_values(self, x, step: StepContext):
+        """(rows for the queries; rows for the values this layer leaves for later ones, or None; those an earlier one left, or None)."""
+        make = torch.zeros if step.padded else torch.empty
+        rows = lambda width: make((step.n_tokens, width), dtype=self.runtime.dtype, device=x.device)
+        keep = first = None
+        if self.value_mix == "keep":
+            keep = step.shared["values"] = rows(self.KV * self.vd)
+        elif self.value_mix == "mix":
+            first = step.shared["values"]
+        return rows(self.H * self.hd), keep, first
+
+    def _forward_own_values(self, x, step: StepContext, cache: CacheView) -> torch.Tensor:
         n, dt = step.n_tokens, self.runtime.dtype
         q = self._prepare(x, step, cache)
         # rows that belong to no sequence (a small step's padding) are not written by the kernels: keep them defined
@@ -240,9 +289,9 @@ class WindowAttentionMixer(Mixer):
                 reach = [-(-int(r) // ops.PAGE) + 1 for r in (self.chunk, window) if r]
                 splits = min([ops.decode_attention_splits(step.n_seqs, self.KV, self.hd, getattr(step, "context_class", 0))] + reach)
             ops.attention_chunked_mma(q, q.stride(0), attn, cache.k, cache.v, cache.block_table, step, self.H, self.KV, self.hd, self.vd,
-                                      self.scale, window=window, chunk=self.chunk, distance_bias=self.distance_bias, splits=splits,
-                                      few_rows=step.is_decode)
+                                      self.scale, window=window, chunk=self.chunk, distance_bias=self.distance_bias, sink=self.sink,
+                                      splits=splits, few_rows=step.is_decode)
         else:
             ops.attention_simt(q, q.stride(0), attn, cache.k, cache.v, cache.block_table, step.positions, step.token_slot, n, self.H, self.KV,
-                               self.hd, self.scale, window, value_dim=self.vd, chunk=self.chunk, distance_bias=self.distance_bias)
+                               self.hd, self.scale, window, value_dim=self.vd, sink=self.sink, chunk=self.chunk, distance_bias=self.distance_bias)
         return self.o.forward(attn, allow_partials=True)
