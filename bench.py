@@ -448,6 +448,21 @@ def vepolix_config(width, layers, heads, kv_heads, head_dim, vocab):
             "layers": [order[i % 4] for i in range(layers)]}
 
 
+def voserax_config(width, layers, heads, kv_heads, head_dim, vocab):
+    """A Voserax model of ``layers`` layers between 4 residual streams: every layer attention with the Llama shape's heads (4 taps on
+    q, k and v, half of every head rotated, a window of 1,024, mixed values); in groups of four the first with a dense
+    feed-forward of the Llama shape's intermediate size, the others with 16 experts of a quarter of it and 2 identity experts of which
+    a token uses 4, and a shared expert of that size."""
+    inter = COMPARE_INTER[width]
+    att = {"type": "attention", "mixer": {"heads": heads, "kv_heads": kv_heads, "dim": head_dim, "vdim": head_dim, "scale": head_dim ** -0.5, "conv": 4,
+                                          "mask": {"size": 1024}, "v_mix": True,
+                                          "rot": {"base": 500000.0, "dims": head_dim // 2, "scaling": {"factor": 8.0, "original": 8192, "fast": 32.0, "slow": 1.0}}}}
+    moe = {"kind": "moe", "router": {"experts": 16, "top": 4, "identity": 2}, "expert": {"ff": inter // 4, "limit": 7.0},
+           "shared": {"ff": inter // 4, "limit": 7.0}}
+    return {"architecture": "Voserax", "vocab": vocab, "width": width, "streams": 4, "residual_mult": 1.0, "norm": {"eps": 1e-5}, "max_positions": 4096,
+            "layers": [dict(att, mlp={"kind": "dense", "ff": inter} if i % 4 == 0 else moe) for i in range(layers)]}
+
+
 COMPARE_INTER = {2048: 8192, 4096: 14336}
 
 
@@ -461,7 +476,7 @@ COMPARE_SIZES = {
 
 
 def compare_designs(args):
-    """``--compare terolix`` (or ``munadra``, ``bededra``, ``dofevik``, ``vepolix``): prefill (one prompt of 2,048 tokens) and decode (8 and 64 sequences after
+    """``--compare terolix`` (or ``munadra``, ``bededra``, ``dofevik``, ``vepolix``, ``voserax``): prefill (one prompt of 2,048 tokens) and decode (8 and 64 sequences after
     512-token prompts, CUDA graphs) of Terolix beside the Llama decoder at equal size, random weights,
     bfloat16.  Rates in tokens a second; ``hbm_frac`` is the weights' bytes over the decode step's time
     over the copy peak, ``tc_frac`` the prefill's matrix-product flops over its time over the bf16 peak."""
@@ -492,18 +507,23 @@ def compare_designs(args):
         if args.compare == "vepolix":                     # beside the closest existing model: matrix recurrences, parallel blocks, grouped experts
             base, llama = "bededra", other
             other = vepolix_config(z["width"], z["layers"], z["heads"], z["kv_heads"], z["head_dim"], vocab)
+        if args.compare == "voserax":                     # beside the closest existing model: windows with a sink, experts with a shared one in every layer
+            base, llama = "dofevik", dofevik_config(z["width"], z["layers"], z["heads"], z["kv_heads"], z["head_dim"], vocab)
+            other = voserax_config(z["width"], z["layers"], z["heads"], z["kv_heads"], z["head_dim"], vocab)
         out[name] = {}
         for design, cfg in ((base, llama), (args.compare, other)):
             model = kl.random_model(config_from_dict(cfg), seed=0, dtype="bfloat16", device="cuda:0")
             infer = kl.Inference(model, max_tokens=64 * CONTEXT, max_batch=64, max_seq_len=CONTEXT)
             wbytes = model.weight_bytes()
             matrix_params = wbytes / 2 - vocab * z["width"]
-            if design in ("munadra", "bededra", "dofevik", "vepolix"):       # a token uses 4 of a layer's 16 experts: count what it multiplies by
+            if design in ("munadra", "bededra", "dofevik", "vepolix", "voserax"):       # a token uses 4 of a layer's 16 experts: count what it multiplies by
                 moe_layers = sum(1 for l in cfg["layers"] if l["mlp"] and l["mlp"]["kind"] == "moe")
                 per_expert = (2 if design == "dofevik" else 3) * z["width"] * (COMPARE_INTER[z["width"]] // 4)   # no gate: two matrices
                 matrix_params -= moe_layers * 12 * per_expert
             if design in ("dofevik", "vepolix"):
                 matrix_params -= vocab * z["width"]           # a classifier of its own, which runs on the wanted rows only
+            if design == "voserax":
+                matrix_params -= cfg["max_positions"] * z["width"]     # position vectors are looked up
             t = time_prefill(infer, warmup=3, repeats=5, seed=2, checks=checks)
             r = {"weight_gb": round(wbytes / 1e9, 3), "prefill_tokens_per_s": round(PREFILL_LEN / t, 1), "prefill_ms": round(t * 1e3, 3),
                  "prefill_tc_frac": round(2 * PREFILL_LEN * matrix_params / t / (pk["bf16_tflops"] * 1e12), 4)}
@@ -551,8 +571,8 @@ def main():
     ap.add_argument("--dtype", default="bfloat16", choices=["bfloat16", "float32"])
     ap.add_argument("--no-points", action="store_true",
                     help="only the headline: skip the prefill, the batch 1, 64 and 128 points and the two other workloads")
-    ap.add_argument("--compare", default=None, choices=["terolix", "munadra", "bededra", "dofevik", "vepolix"],
-                    help="instead of the default workload: this design beside Llama (Dofevik: beside Munadra, Vepolix: beside Bededra) at equal size (prefill and decode rates)")
+    ap.add_argument("--compare", default=None, choices=["terolix", "munadra", "bededra", "dofevik", "vepolix", "voserax"],
+                    help="instead of the default workload: this design beside Llama (Dofevik: beside Munadra, Vepolix: beside Bededra, Voserax: beside Dofevik) at equal size (prefill and decode rates)")
     ap.add_argument("--sizes", default="", help="with --compare: which of the sizes to run, with commas (default: all)")
     args = ap.parse_args()
     if args.impl == "reference":

@@ -33,7 +33,8 @@ KERNEL_ENTRY_POINTS = ("embedding", "add_rmsnorm", "swiglu", "rope_kv_write", "a
                        "gemm_skinny_partials", "gemm_skinny", "attention_decode", "attention_mma", "attention_tcgen05",
                        "attention_decode_fused", "norm_chain", "head_rmsnorm_gate", "activation", "sigmoid_gate", "mingru_scan",
                        "gated_delta_rule", "grouped_gemm", "grouped_gemv", "gemm_tcgen05_grouped", "gemm_tcgen05_grouped_skinny", "moe_route", "moe_plan", "moe_gather", "moe_combine",
-                       "latent_prepare", "latent_attention", "causal_conv", "rglru_gate", "linear_scan")
+                       "latent_prepare", "latent_attention", "causal_conv", "rglru_gate", "linear_scan", "pair_rmsnorm", "stream_norm", "qk_prepare",
+                       "qk_row_prepare", "qkv_conv", "attention_chunked_mma", "short_conv")
 
 
 class KernelTimes:
