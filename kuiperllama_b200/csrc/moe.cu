@@ -200,18 +200,19 @@ struct CombineArgs {
     float* out;
 };
 
-// V elements of a row a thread (V = 16 bytes of results an access where rows allow it, else 1), a token's results on their way four
-// at a time.
-template <typename T, int V> __device__ __forceinline__ void mc_load(const T* p, float (&x)[V]) {
-    if constexpr (V == 1) x[0] = to_f32(p[0]);
-    else {
-        const uint4 raw = *reinterpret_cast<const uint4*>(p);
-        const T* e = reinterpret_cast<const T*>(&raw);
+// V elements of a row a thread (16 bytes of results an access where rows allow it; with PIECES, few rows, 4 elements, so that
+// more threads share them; else 1), a token's results on their way four at a time, pieces eight at a time and ahead of them.
+template <typename T, int V> struct McRaw { T v[V]; };       // a piece of a row as it lies in memory, held while it is on its way
+template <> struct McRaw<bf16, 8> { uint4 v; };
+template <> struct McRaw<bf16, 4> { uint2 v; };
+template <> struct McRaw<float, 4> { uint4 v; };
+template <typename T, int V> __device__ __forceinline__ McRaw<T, V> mc_fetch(const T* p) { return *reinterpret_cast<const McRaw<T, V>*>(p); }
+template <typename T, int V> __device__ __forceinline__ void mc_axpy(float a, const McRaw<T, V>& raw, float (&acc)[V]) {
+    const T* e = reinterpret_cast<const T*>(&raw);
 #pragma unroll
-        for (int i = 0; i < V; ++i) x[i] = to_f32(e[i]);
-    }
+    for (int i = 0; i < V; ++i) acc[i] = fmaf(a, to_f32(e[i]), acc[i]);
 }
-template <typename T, int V>
+template <typename T, int V, bool PIECES>
 __global__ void __launch_bounds__(256)
 moe_combine_kernel(const CombineArgs A) {
     pdl_launch_dependents();
@@ -221,46 +222,48 @@ moe_combine_kernel(const CombineArgs A) {
     for (size_t idx = (size_t)blockIdx.x * blockDim.x + threadIdx.x; idx < total; idx += (size_t)gridDim.x * blockDim.x) {
         const size_t t = idx / per;
         const int c = (int)(idx - t * per) * V;
-        float acc[V];
+        float acc[V], y[V];
 #pragma unroll
-        for (int e = 0; e < V; ++e) acc[e] = 0.f;
+        for (int e = 0; e < V; ++e) acc[e] = y[e] = 0.f;
+        // the expert every token takes: its result is asked for first and joins the sum last
+        McRaw<T, V> every;
+        if (!PIECES && A.shared != nullptr) every = mc_fetch<T, V>((const T*)A.shared + t * A.shared_ld + c);
+        const float z_gate = A.gate != nullptr ? A.gate[t * A.gate_ld] : 0.f;
+        if constexpr (PIECES) {
+            const float* p = A.pieces + t * A.hidden + c;
+            for (int z0 = 0; z0 < A.n_pieces; z0 += 8) {                 // pieces are added in ascending order
+                McRaw<float, V> q[8];
+#pragma unroll
+                for (int z = 0; z < 8; ++z)
+                    if (z0 + z < A.n_pieces) q[z] = mc_fetch<float, V>(p + (size_t)(z0 + z) * A.piece_stride);
+#pragma unroll
+                for (int z = 0; z < 8; ++z)
+                    if (z0 + z < A.n_pieces) mc_axpy<float, V>(1.0f, q[z], y);
+            }
+        }
         for (int k0 = 0; k0 < top; k0 += 4) {
-            float r[4][V], wt[4];
+            McRaw<T, V> r[4];
+            float wt[4];
+            bool any[4];
 #pragma unroll
             for (int k = 0; k < 4; ++k) {
                 const int pos = k0 + k < top ? A.pair_pos[t * top + k0 + k] : -1;
                 const T* src = pos >= 0 ? (const T*)A.results + (size_t)pos * A.ld + c
                                         : (pos == -2 && A.x != nullptr ? (const T*)A.x + t * A.x_ld + c : nullptr);
-                wt[k] = src != nullptr ? A.weight[t * top + k0 + k] : 0.f;
-                if (src != nullptr) mc_load<T, V>(src, r[k]);
-                else {
-#pragma unroll
-                    for (int e = 0; e < V; ++e) r[k][e] = 0.f;
-                }
+                any[k] = src != nullptr;
+                wt[k] = any[k] ? A.weight[t * top + k0 + k] : 0.f;
+                if (any[k]) r[k] = mc_fetch<T, V>(src);
             }
 #pragma unroll
             for (int k = 0; k < 4; ++k)
-#pragma unroll
-                for (int e = 0; e < V; ++e) acc[e] = fmaf(wt[k], r[k][e], acc[e]);
+                if (any[k]) mc_axpy<T, V>(wt[k], r[k], acc);
         }
-        if (A.shared != nullptr || A.n_pieces > 0) {
-            float y[V];
+        if (PIECES || A.shared != nullptr) {
+            const float f = A.gate != nullptr ? 1.0f / (1.0f + expf(-z_gate)) : 1.0f;
+            if constexpr (PIECES) {
 #pragma unroll
-            for (int e = 0; e < V; ++e) y[e] = 0.f;
-            if (A.shared != nullptr) mc_load<T, V>((const T*)A.shared + t * A.shared_ld + c, y);
-            for (int z = 0; z < A.n_pieces; ++z) {
-                const float* p = A.pieces + (size_t)z * A.piece_stride + t * A.hidden + c;
-                if constexpr (V % 4 == 0) {
-#pragma unroll
-                    for (int e = 0; e < V; e += 4) {
-                        const float4 q = *reinterpret_cast<const float4*>(p + e);
-                        y[e] += q.x; y[e + 1] += q.y; y[e + 2] += q.z; y[e + 3] += q.w;
-                    }
-                } else y[0] += p[0];
-            }
-            const float f = A.gate != nullptr ? 1.0f / (1.0f + expf(-A.gate[t * A.gate_ld])) : 1.0f;
-#pragma unroll
-            for (int e = 0; e < V; ++e) acc[e] = fmaf(f, y[e], acc[e]);
+                for (int e = 0; e < V; ++e) acc[e] = fmaf(f, y[e], acc[e]);
+            } else mc_axpy<T, V>(f, every, acc);
         }
         float* o = A.out + t * A.hidden + c;
         if constexpr (V % 4 == 0) {
@@ -340,17 +343,20 @@ KL_API int kl_moe_combine(const void* results, long long ld, const int* pair_pos
     if (dtype != KL_F32 && dtype != KL_BF16) return KL_ERR_BAD_DTYPE;
     if (n_pieces < 0 || (n_pieces > 0 && (pieces == nullptr || shared != nullptr))) return KL_ERR_BAD_SIZE;
     const CombineArgs A{results, ld, pair_pos, weight, x, x_ld, shared, shared_ld, pieces, n_pieces, piece_stride, gate, gate_ld, tokens, top, hidden, out};
-    const int v = dtype == KL_F32 ? 4 : 8;
+    const int v = (dtype == KL_F32 || n_pieces > 0) ? 4 : 8;
     const bool wide = hidden % v == 0 && ld % v == 0 && x_ld % v == 0 && shared_ld % v == 0 && piece_stride % v == 0 &&
                       (((uintptr_t)results | (uintptr_t)out | (uintptr_t)x | (uintptr_t)shared | (uintptr_t)pieces) & 15) == 0;
-    const int grid = kl::strided_grid((size_t)tokens * (wide ? hidden / v : hidden), 256, 16);
+    const int threads = n_pieces > 0 ? 128 : 256;
+    const int grid = kl::strided_grid((size_t)tokens * (wide ? hidden / v : hidden), threads, 16);
+#define KL_MC(T, V, P) launch_kernel(moe_combine_kernel<T, V, P>, grid, threads, 0, stream, A)
     if (dtype == KL_F32) {
-        if (wide) launch_kernel(moe_combine_kernel<float, 4>, grid, 256, 0, stream, A);
-        else launch_kernel(moe_combine_kernel<float, 1>, grid, 256, 0, stream, A);
+        if (n_pieces > 0) { if (wide) KL_MC(float, 4, true); else KL_MC(float, 1, true); }
+        else { if (wide) KL_MC(float, 4, false); else KL_MC(float, 1, false); }
     } else {
-        if (wide) launch_kernel(moe_combine_kernel<bf16, 8>, grid, 256, 0, stream, A);
-        else launch_kernel(moe_combine_kernel<bf16, 1>, grid, 256, 0, stream, A);
+        if (n_pieces > 0) { if (wide) KL_MC(bf16, 4, true); else KL_MC(bf16, 1, true); }
+        else { if (wide) KL_MC(bf16, 8, false); else KL_MC(bf16, 1, false); }
     }
+#undef KL_MC
     KL_LAUNCH_CHECK();
     return KL_OK;
 }

@@ -94,15 +94,16 @@ stream_norm_vec_kernel(const StreamNorm A) {
         if (update) {
             float4 y = make_float4(0.f, 0.f, 0.f, 0.f);
             if (d != nullptr) y = Quad<T>::load(d + 4 * i4);
-            // four pieces are requested at a time and added in ascending order
-            for (int z0 = 0; z0 < A.n_pieces; z0 += 4) {
-                float4 b[4];
+            // four pieces (eight in the form for few rows) are requested at a time and added in ascending order
+            constexpr int ZB = THREADS == 512 && VPT == 1 ? 8 : 4;
+            for (int z0 = 0; z0 < A.n_pieces; z0 += ZB) {
+                float4 b[ZB];
 #pragma unroll
-                for (int z = 0; z < 4; ++z)
+                for (int z = 0; z < ZB; ++z)
                     b[z] = z0 + z < A.n_pieces ? *reinterpret_cast<const float4*>(p + (size_t)(z0 + z) * A.piece_stride + 4 * i4)
                                                : make_float4(0.f, 0.f, 0.f, 0.f);
 #pragma unroll
-                for (int z = 0; z < 4; ++z) { y.x += b[z].x; y.y += b[z].y; y.z += b[z].z; y.w += b[z].w; }
+                for (int z = 0; z < ZB; ++z) { y.x += b[z].x; y.y += b[z].y; y.z += b[z].z; y.w += b[z].w; }
             }
             float4 n[S];
 #pragma unroll
