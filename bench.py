@@ -4,8 +4,9 @@ B200, and the two other workloads of the same family (Llama-2-7B shape with ragg
 Llama-3.2-1B shape with temperature sampling).
 
     python bench.py [--gpus 1] [--steps K] [--warmup W] [--layers L] [--batch B] [--impl reference] [--no-points]
-    python bench.py --compare terolix|munadra|bededra|dofevik|vepolix [--sizes 1b,8b-8-layers]   (another design beside Llama, or beside the
-                                                 closest model: Dofevik beside Munadra, Vepolix beside Bededra; see compare_designs)
+    python bench.py --compare terolix|munadra|bededra|dofevik|vepolix|voserax [--sizes 1b,8b-8-layers]   (another design beside Llama, or beside the
+                                                 closest model: Dofevik beside Munadra, Vepolix beside Bededra, Voserax beside
+                                                 Dofevik; see compare_designs)
 
 A "step" is one decode step of a batch (default 8 sequences that each hold a 512-token
 prompt, context limit 4096).  One JSON line is printed:
